@@ -77,12 +77,16 @@ class ModelSpec:
     order: List[RunSpec]
     final_norm: PartSpec
     head: PartSpec
+    # the residual stream as several copies that every block mixes ([T, streams, hidden]; its blocks say so too); None: one stream
+    streams: Optional[int] = None
     # names a checkpoint may carry although no part asks for them (tensors of a sub-layer that a layer leaves out)
     tolerated_tensors: tuple = ()
 
     def validate(self) -> None:
         if self.hidden_size <= 0 or self.vocab_size <= 0 or self.max_position <= 0:
             raise ValueError("hidden_size, vocab_size and max_position must be positive")
+        if self.streams is not None and self.streams <= 0:
+            raise ValueError("streams must be positive")
         if not self.layers or not self.order:
             raise ValueError("a model needs at least one layer and one run")
         for i, run in enumerate(self.order):

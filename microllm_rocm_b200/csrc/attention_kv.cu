@@ -13,7 +13,8 @@
 //                           32 at absolute multiples of 32 with a running maximum and sum (the order of every addition
 //                           depends on the position alone, not on how the tokens were cut into steps), optional window,
 //                           optional output gate: o * sigmoid(gate) with the gate read from a projection's fp32 output
-//                           (one gate per element of a head, or one per head); optional cap on the scores,
+//                           (one gate per element of a head, or one per head); optional bias per head and distance
+//                           query - key, added to the scaled score; optional cap on the scores,
 //                           s <- cap * tanh(s / cap); optional sink: exp(sink[head]) joins the softmax's denominator
 //                           (no key, no value, neither scaled nor capped).
 //
@@ -155,6 +156,7 @@ struct AttnParams {
     int gate_per_head;               // 1: one gate per (token, head) at gate_col + head; 0: one per element at gate_col + head * dv + c
     const float* sink;               // [heads] or null: exp(sink[head]) joins the denominator
     float softcap;                   // > 0: s <- softcap * tanh(s / softcap)
+    DistanceBias bias;               // added to the scaled (and capped) score
     int* error_flag;
 };
 
@@ -186,6 +188,7 @@ __global__ void __launch_bounds__(WARPS * 32) paged_attention_kv_kernel(AttnPara
     const size_t v_base = (size_t)p.num_kv_heads * p.page_size * DK;
     const int* table = p.block_table + (size_t)seq * p.max_blocks;
 
+    const float* const bias_row = p.bias.table ? p.bias.row(h) : nullptr;
     for (int base = (lo / 32) * 32; base <= pos; base += 32) {
         const int kp = base + lane;
         bool valid = kp >= lo && kp <= pos;
@@ -209,6 +212,7 @@ __global__ void __launch_bounds__(WARPS * 32) paged_attention_kv_kernel(AttnPara
             for (int c = 0; c < DK; ++c) dot = fmaf(q_s[warp][c], to_f32(krow[c]), dot);
             s = dot * p.scale;
             if (p.softcap > 0.0f) s = p.softcap * tanhf(s / p.softcap);
+            if (bias_row) s += p.bias.at(bias_row, pos - kp);
         }
         const float m_new = fmaxf(m, warp_max(s));
         if (m_new == -INFINITY) continue;
@@ -410,7 +414,7 @@ MLB_EXPORT int mlb_paged_attention_kv(const void* q, int q_dtype, const void* pa
                                       int num_pages, int page_size, int tokens, int num_heads, int num_kv_heads, int dk, int dv,
                                       int window, int chunk, float scale, const float* gate, long long gate_ld, int gate_partials,
                                       long long gate_partial_stride, int gate_col, int gate_per_head, const float* sink, float softcap,
-                                      int* error_flag, cudaStream_t stream) {
+                                      const float* distance_bias, int last_distance, int* error_flag, cudaStream_t stream) {
     if (tokens < 0 || num_heads <= 0 || num_kv_heads <= 0 || num_heads % num_kv_heads != 0)
         return fail(MLB_INVALID_ARGUMENT, "paged_attention_kv: bad head counts %d/%d", num_heads, num_kv_heads);
     if (dk <= 0 || dk > MAX_D || dv <= 0 || dv > MAX_D)
@@ -420,7 +424,8 @@ MLB_EXPORT int mlb_paged_attention_kv(const void* q, int q_dtype, const void* pa
     if (tokens == 0) return MLB_OK;
     AttnParams p{q, pages, out, positions, token_seq, block_table, max_blocks, num_pages, page_size, tokens, num_heads,
                  num_kv_heads, dk, dv, chunk, window, scale, Columns{gate, gate_ld, gate_partials < 1 ? 1 : gate_partials, gate_partial_stride},
-                 gate_col, gate_per_head ? 1 : 0, sink, softcap, error_flag};
+                 gate_col, gate_per_head ? 1 : 0, sink, softcap, DistanceBias{distance_bias, last_distance}, error_flag};
+    if (distance_bias && last_distance < 0) return fail(MLB_INVALID_ARGUMENT, "paged_attention_kv: a distance bias has a last distance");
     if (softcap < 0.0f) return fail(MLB_INVALID_ARGUMENT, "paged_attention_kv: a cap on the scores is positive (0: none)");
     const long long items = (long long)tokens * num_heads;
     const unsigned blocks = (unsigned)((items + WARPS - 1) / WARPS);

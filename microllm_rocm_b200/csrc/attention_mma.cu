@@ -69,6 +69,7 @@ struct FaParams {
                                     // portions), 0 = work item i is sequence i and token i (every sequence brings one token)
     float cap_pre;                  // > 0: scores are capped, s <- cap * tanh(s * scale / cap); this is scale / cap
     const float* sink;              // [num_heads] or null: exp(sink[head]) joins the head's denominator (no key, no value)
+    DistanceBias bias;              // added to the scaled (and capped) score
 };
 
 __device__ __forceinline__ void mma_bf16(float (&c)[4], unsigned a0, unsigned a1, unsigned a2, unsigned a3,
@@ -101,6 +102,11 @@ __device__ __forceinline__ float fast_tanh(float x) {
 // a raw dot product -> the score in base-2 units: s * scale * log2(e), or with a cap: cap * tanh(s * scale / cap) * log2(e)
 __device__ __forceinline__ float score_log2(const FaParams& p, float s) {
     return (p.cap_pre > 0.0f ? fast_tanh(s * p.cap_pre) : s) * p.scale_log2;
+}
+// the same with the bias of a distance (row: the head's values, null without a bias)
+__device__ __forceinline__ float score_log2(const FaParams& p, float s, const float* row, int distance) {
+    const float v = score_log2(p, s);
+    return row ? fmaf(p.bias.at(row, distance), LOG2E, v) : v;
 }
 // What the accumulator of a row is multiplied by at the end: 1 / l, or with a sink 1 / (l + 2^(sink log2 e - m)), where the
 // row's sum l and its accumulator are relative to 2^m (m in base-2 units; -inf: the row saw no key).
@@ -214,8 +220,8 @@ __device__ __forceinline__ void load_keys(const FaParams& p, const TileGeometry&
 // One 16-key tile through scores, running softmax and the value product.
 // first_pos: the smallest position of any real row of the row tile; last_lo: the largest window start.
 __device__ __forceinline__ void consume_keys(const FaParams& p, const __nv_bfloat16* q_s, const KeyTile& kv,
-                                             const int (&pos_row)[2], const int (&lo_row)[2], int first_pos, int last_lo,
-                                             RowState& st) {
+                                             const int (&pos_row)[2], const int (&lo_row)[2], const float* const (&bias_row)[2],
+                                             int first_pos, int last_lo, RowState& st) {
     if (kv.base < 0) return;
     const int lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
     float s[2][4];
@@ -245,7 +251,7 @@ __device__ __forceinline__ void consume_keys(const FaParams& p, const __nv_bfloa
                 const int i = e >> 1;
                 const int key = kv.base + nb * 8 + 2 * t + (e & 1);
                 const bool ok = key >= lo_row[i] && key <= pos_row[i];
-                s[nb][e] = ok ? score_log2(p, s[nb][e]) : -INFINITY;
+                s[nb][e] = ok ? score_log2(p, s[nb][e], bias_row[i], pos_row[i] - key) : -INFINITY;
                 mx[i] = fmaxf(mx[i], s[nb][e]);
             }
     } else {
@@ -253,7 +259,7 @@ __device__ __forceinline__ void consume_keys(const FaParams& p, const __nv_bfloa
         for (int nb = 0; nb < 2; ++nb)
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
-                s[nb][e] = score_log2(p, s[nb][e]);
+                s[nb][e] = score_log2(p, s[nb][e], bias_row[e >> 1], pos_row[e >> 1] - (kv.base + nb * 8 + 2 * t + (e & 1)));
                 mx[e >> 1] = fmaxf(mx[e >> 1], s[nb][e]);
             }
     }
@@ -336,6 +342,9 @@ __device__ __forceinline__ void attend(const FaParams& p, const TileGeometry& ge
             lo_row[i] = 0;
         }
     }
+    const float* bias_row[2];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) bias_row[i] = p.bias.table ? p.bias.row(geo.kvh * p.group + (geo.row0 + g + 8 * i) % p.group) : nullptr;
     int first_pos = 0x7fffffff, last_lo = 0;
 #pragma unroll
     for (int i = 0; i < 2; ++i)
@@ -353,12 +362,12 @@ __device__ __forceinline__ void attend(const FaParams& p, const TileGeometry& ge
             const bool more_b = kt + stride < tile_end;
             if (more_b && in_flight < 2) load_keys(p, geo, pt, kt + stride, hi_tile, b);
             in_flight = 0;
-            consume_keys(p, q_s, a, pos_row, lo_row, first_pos, last_lo, st);
+            consume_keys(p, q_s, a, pos_row, lo_row, bias_row, first_pos, last_lo, st);
             if (!more_b) break;
             kt += stride;
             const bool more_a = kt + stride < tile_end;
             if (more_a) load_keys(p, geo, pt, kt + stride, hi_tile, a);
-            consume_keys(p, q_s, b, pos_row, lo_row, first_pos, last_lo, st);
+            consume_keys(p, q_s, b, pos_row, lo_row, bias_row, first_pos, last_lo, st);
             if (!more_a) break;
             kt += stride;
         }
@@ -366,7 +375,7 @@ __device__ __forceinline__ void attend(const FaParams& p, const TileGeometry& ge
         for (; kt < tile_end; kt += stride) {
             if (in_flight < 1) load_keys(p, geo, pt, kt, hi_tile, a);
             in_flight = 0;
-            consume_keys(p, q_s, a, pos_row, lo_row, first_pos, last_lo, st);
+            consume_keys(p, q_s, a, pos_row, lo_row, bias_row, first_pos, last_lo, st);
         }
     }
 }
@@ -513,6 +522,9 @@ __global__ void __launch_bounds__(WARPS * 32, 2) fa_prefill_kernel(FaParams p) {
             lo_row[i] = 0;
         }
     }
+    const float* bias_row[2];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) bias_row[i] = p.bias.table ? p.bias.row(geo.kvh * p.group + (geo.row0 + g + 8 * i) % p.group) : nullptr;
     // the warp's own key range: tiles outside it are skipped (it still keeps step with the CTA)
     const int warp_first_pos = geo.pos0 + geo.token_of(0, p.group);
     const int warp_last_pos = geo.pos0 + min(geo.token_of(15, p.group), geo.n_new - 1);
@@ -576,7 +588,7 @@ __global__ void __launch_bounds__(WARPS * 32, 2) fa_prefill_kernel(FaParams p) {
                 for (int nb = 0; nb < 8; ++nb)
 #pragma unroll
                     for (int e = 0; e < 4; ++e) {
-                        s[nb][e] = score_log2(p, s[nb][e]);
+                        s[nb][e] = score_log2(p, s[nb][e], bias_row[e >> 1], pos_row[e >> 1] - (base + nb * 8 + 2 * t + (e & 1)));
                         mx[e >> 1] = fmaxf(mx[e >> 1], s[nb][e]);
                     }
             } else {
@@ -587,7 +599,7 @@ __global__ void __launch_bounds__(WARPS * 32, 2) fa_prefill_kernel(FaParams p) {
                         const int i = e >> 1;
                         const int key = base + nb * 8 + 2 * t + (e & 1);
                         const bool ok = key >= lo_row[i] && key <= pos_row[i];
-                        s[nb][e] = ok ? score_log2(p, s[nb][e]) : -INFINITY;
+                        s[nb][e] = ok ? score_log2(p, s[nb][e], bias_row[i], pos_row[i] - key) : -INFINITY;
                         mx[i] = fmaxf(mx[i], s[nb][e]);
                     }
             }
@@ -863,7 +875,7 @@ __device__ __forceinline__ int k_column(int c, int t) {
 
 template <bool INTERLEAVED = false>
 __device__ __forceinline__ void consume_keys_t(const FaParams& p, const __nv_bfloat16* q_s, const KeyTile& kv, int last_pos,
-                                               int lo, RowStateT& st) {
+                                               int lo, const float* const (&bias_row)[2], RowStateT& st) {
     if (kv.base < 0) return;
     const int lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
     float s0[4] = {0.0f, 0.0f, 0.0f, 0.0f}, s1[4] = {0.0f, 0.0f, 0.0f, 0.0f};     // two chains
@@ -876,7 +888,7 @@ __device__ __forceinline__ void consume_keys_t(const FaParams& p, const __nv_bfl
     // s[0], s[1]: key base + g, heads 2t, 2t+1;   s[2], s[3]: key base + g + 8
     float s[4];
 #pragma unroll
-    for (int e = 0; e < 4; ++e) s[e] = score_log2(p, s0[e] + s1[e]);
+    for (int e = 0; e < 4; ++e) s[e] = score_log2(p, s0[e] + s1[e], bias_row[e & 1], last_pos - (kv.base + g + 8 * (e >> 1)));
     if (kv.base + 15 > last_pos || kv.base < lo) {         // an edge tile (uniform over the warp)
         const int key0 = kv.base + g, key1 = key0 + 8;
         if (key0 < lo || key0 > last_pos) s[0] = s[1] = -INFINITY;
@@ -938,6 +950,13 @@ __device__ __forceinline__ void consume_keys_t(const FaParams& p, const __nv_bfl
             mma_bf16(st.o[pp * 8 + j], a0, a1, a2, a3, b0, b1);
         }
     }
+}
+
+// the biases by distance of heads 2t and 2t + 1 of a group (a column without a head takes the last head's: its scores are never stored)
+__device__ __forceinline__ void bias_rows_t(const FaParams& p, int kvh, const float* (&bias_row)[2]) {
+    const int t = threadIdx.x & 3;
+#pragma unroll
+    for (int i = 0; i < 2; ++i) bias_row[i] = p.bias.table ? p.bias.row(kvh * p.group + min(2 * t + i, p.group - 1)) : nullptr;
 }
 
 // What follows the key loop of the keys-on-M decode kernels: the warps of a CTA merge their shares in shared
@@ -1103,6 +1122,8 @@ __global__ void __launch_bounds__(DW * 32, DW == 4 ? 2 : 1) fa_decode_t_kernel(F
     for (int k = 0; k < NPAIR * 8; ++k)
 #pragma unroll
         for (int e = 0; e < 4; ++e) st.o[k][e] = 0.0f;
+    const float* bias_row[2];
+    bias_rows_t(p, geo.kvh, bias_row);
     if (kt < tile_end) {
         if (USE_PREFETCH) {
             if (in_flight < 1) load_keys(p, geo, pt, kt, last_pos, tile_a);
@@ -1110,12 +1131,12 @@ __global__ void __launch_bounds__(DW * 32, DW == 4 ? 2 : 1) fa_decode_t_kernel(F
                 const bool more_b = kt + DW < tile_end;
                 if (more_b && in_flight < 2) load_keys(p, geo, pt, kt + DW, last_pos, tile_b);
                 in_flight = 0;
-                consume_keys_t(p, q_s, tile_a, last_pos, lo, st);
+                consume_keys_t(p, q_s, tile_a, last_pos, lo, bias_row, st);
                 if (!more_b) break;
                 kt += DW;
                 const bool more_a = kt + DW < tile_end;
                 if (more_a) load_keys(p, geo, pt, kt + DW, last_pos, tile_a);
-                consume_keys_t(p, q_s, tile_b, last_pos, lo, st);
+                consume_keys_t(p, q_s, tile_b, last_pos, lo, bias_row, st);
                 if (!more_a) break;
                 kt += DW;
             }
@@ -1123,7 +1144,7 @@ __global__ void __launch_bounds__(DW * 32, DW == 4 ? 2 : 1) fa_decode_t_kernel(F
             for (; kt < tile_end; kt += DW) {
                 if (in_flight < 1) load_keys(p, geo, pt, kt, last_pos, tile_a);
                 in_flight = 0;
-                consume_keys_t(p, q_s, tile_a, last_pos, lo, st);
+                consume_keys_t(p, q_s, tile_a, last_pos, lo, bias_row, st);
             }
         }
     }
@@ -1262,6 +1283,8 @@ __global__ void __launch_bounds__(160, 2) fa_decode_ring_kernel(const __grid_con
     for (int k = 0; k < NPAIR * 8; ++k)
 #pragma unroll
         for (int e = 0; e < 4; ++e) st.o[k][e] = 0.0f;
+    const float* bias_row[2];
+    bias_rows_t(p, geo.kvh, bias_row);
 
     if (warp == DW) {
         // ---------------------------------------------------------------- the copying warp
@@ -1343,7 +1366,7 @@ __global__ void __launch_bounds__(160, 2) fa_decode_ring_kernel(const __grid_con
             }
             __syncwarp();
             if (lane == 0) mbar_arrive(smem_u32(&empty_bar[s]));      // the stage may be refilled while this tile is used
-            consume_keys_t<true>(p, q_s, tile, last_pos, lo, st);
+            consume_keys_t<true>(p, q_s, tile, last_pos, lo, bias_row, st);
         }
         asm volatile("bar.sync 1, 128;" ::: "memory");          // every warp has taken its last tile: the ring may become the merge's scratch
     }
@@ -1410,7 +1433,7 @@ MLB_EXPORT int mlb_paged_attention_mma(const void* q, const void* pages, void* o
                                        const int* seq_pos0, const int* block_table, const int* work, int num_work,
                                        int max_blocks, int num_pages, int page_size, int num_heads, int num_kv_heads,
                                        int window, int chunk, float scale, int mode, int splits, const float* sink, float softcap,
-                                       int* error_flag, cudaStream_t stream) {
+                                       const float* distance_bias, int last_distance, int* error_flag, cudaStream_t stream) {
     if (num_heads <= 0 || num_kv_heads <= 0 || num_heads % num_kv_heads != 0)
         return fail(MLB_INVALID_ARGUMENT, "paged_attention_mma: bad head counts %d/%d", num_heads, num_kv_heads);
     if (page_size <= 0 || page_size % 16 != 0)
@@ -1430,7 +1453,8 @@ MLB_EXPORT int mlb_paged_attention_mma(const void* q, const void* pages, void* o
                block_table, work, max_blocks, num_pages, page_size, num_heads, num_kv_heads,
                num_heads / num_kv_heads, chunk, window, softcap > 0.0f ? softcap * LOG2E : scale * LOG2E,
                (page_size & (page_size - 1)) == 0 ? __builtin_ctz((unsigned)page_size) : -1, error_flag,
-               mode == 2 ? 1 : 0, softcap > 0.0f ? scale / softcap : 0.0f, sink};
+               mode == 2 ? 1 : 0, softcap > 0.0f ? scale / softcap : 0.0f, sink, DistanceBias{distance_bias, last_distance}};
+    if (distance_bias && last_distance < 0) return fail(MLB_INVALID_ARGUMENT, "paged_attention_mma: a distance bias has a last distance");
     if (mode == 0) {
         static bool prefill_configured_on[MAX_DEVICES] = {false};
         bool& prefill_configured = prefill_configured_on[device_index()];

@@ -24,6 +24,8 @@
 //                P and the row sum use the same (stale) reference, so the quotient is exact.
 //                V rows of keys that no row of the tile may see are cleared in shared memory, so
 //                that whatever an unused slot of a page holds cannot reach the output.
+// A bias by distance joins the scores behind the tensor core: score by score in the tiles near the diagonal, as one number in the
+// tiles whose distances all lie beyond the table's last one.
 // V is used as stored, [key, head element]: it is the MN-major B operand of P V.
 //
 // Formulas as the plain kernel's (attention_plain.cu; src/ops/ops.cpp:2343-2384 in the
@@ -79,6 +81,7 @@ struct TcParams {
     int* error_flag;
     float cap_pre;                  // > 0: scores are capped, s <- cap * tanh(s * scale / cap); this is scale / cap
     const float* sink;              // [num_heads] or null: exp(sink[head]) joins the head's denominator (no key, no value)
+    DistanceBias bias;              // added to the scaled (and capped) score
 };
 
 __device__ __forceinline__ uint32_t smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
@@ -404,6 +407,23 @@ fa_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_con
                 }
             }
             const int kbase = (kt_begin + j) * BN;
+            // a bias by distance: one number for a tile all of whose distances lie at or beyond the table's last one, else
+            // it is added score by score (in base-2 units, so that scale and offset below are 1 and 0)
+            float sc = p.scale_log2, off = 0.0f;
+            if (p.bias.table) {
+                const float* const by_distance = p.bias.row(head);
+                if (qpos_first - (kbase + BN - 1) >= p.bias.last) {
+                    off = by_distance[p.bias.last] * LOG2E;
+                } else {
+                    // distances of this tile: qpos_first - kbase - (BN - 1) .. qpos_first - kbase + BM - 1; the padding in
+                    // front and behind covers what lies outside 0 .. last
+                    const float* const mine = by_distance + (qpos - kbase);
+#pragma unroll
+                    for (int c = 0; c < BN; ++c)
+                        sr[c] = __float_as_uint(fmaf(__uint_as_float(sr[c]), sc, __ldg(mine - c) * LOG2E));
+                    sc = 1.0f;
+                }
+            }
             const bool edge = (kbase + BN - 1 > qpos_first) || (kbase < first_visible_key(qpos_last, p.window, p.chunk));
             float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};       // four chains: no 128-long dependence
             if (edge) {
@@ -419,7 +439,7 @@ fa_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_con
                 for (int c = 0; c < BN; ++c) mx4[c & 3] = fmaxf(mx4[c & 3], __uint_as_float(sr[c]));
             }
             const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
-            const float m_new = fmaxf(m_used, mx * p.scale_log2);
+            const float m_new = fmaxf(m_used, fmaf(mx, sc, off));
             const bool grow = m_new > m_used + RESCALE_STEP;          // also true for the first finite maximum
             const float alpha = grow ? (m_used == -INFINITY ? 0.0f : fast_exp2(m_used - m_new)) : 1.0f;
             if (j > 0 && __any_sync(0xffffffffu, grow)) {
@@ -439,13 +459,14 @@ fa_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_con
             }
             if (grow) { l *= alpha; m_used = m_new; }
             const float m_ref = m_used == -INFINITY ? 0.0f : m_used;
-            // P = 2^(s * scale - m), rounded to bf16 for the tensor core; the sum keeps fp32 terms
+            const float shift = off - m_ref;
+            // P = 2^(s * scale + bias - m), rounded to bf16 for the tensor core; the sum keeps fp32 terms
             float sum4[4] = {0.0f, 0.0f, 0.0f, 0.0f};
             uint32_t packed[BN / 2];
 #pragma unroll
             for (int c = 0; c < BN; c += 2) {
-                const float p0 = fast_exp2(fmaf(__uint_as_float(sr[c]), p.scale_log2, -m_ref));
-                const float p1 = fast_exp2(fmaf(__uint_as_float(sr[c + 1]), p.scale_log2, -m_ref));
+                const float p0 = fast_exp2(fmaf(__uint_as_float(sr[c]), sc, shift));
+                const float p1 = fast_exp2(fmaf(__uint_as_float(sr[c + 1]), sc, shift));
                 sum4[(c >> 1) & 3] += p0 + p1;
                 packed[c / 2] = pack_bf16(p0, p1);
             }
@@ -577,7 +598,7 @@ MLB_EXPORT int mlb_paged_attention_tc(const void* q, long long ldq, const void* 
                                       const int* seq_starts, const int* seq_pos0, const int* block_table, const int* work,
                                       int num_work, int max_blocks, int num_pages, int page_size, int num_heads,
                                       int num_kv_heads, int window, int chunk, float scale, const float* sink, float softcap,
-                                      int* error_flag, cudaStream_t stream) {
+                                      const float* distance_bias, int last_distance, int* error_flag, cudaStream_t stream) {
     if (num_heads <= 0 || num_kv_heads <= 0 || num_heads % num_kv_heads != 0)
         return fail(MLB_INVALID_ARGUMENT, "attention_tc: bad head counts %d/%d", num_heads, num_kv_heads);
     if (!mlb_fa_tc_supported(page_size, scale)) return MLB_UNSUPPORTED_SIZE;
@@ -599,7 +620,9 @@ MLB_EXPORT int mlb_paged_attention_tc(const void* q, long long ldq, const void* 
 
     TcParams p{(__nv_bfloat16*)out, ldo, seq_starts, seq_pos0, block_table, work, max_blocks, num_pages, page_size,
                BN / page_size, num_heads, num_kv_heads, num_heads / num_kv_heads, window, chunk,
-               softcap > 0.0f ? softcap * LOG2E : scale * LOG2E, error_flag, softcap > 0.0f ? scale / softcap : 0.0f, sink};
+               softcap > 0.0f ? softcap * LOG2E : scale * LOG2E, error_flag, softcap > 0.0f ? scale / softcap : 0.0f, sink,
+               DistanceBias{distance_bias, last_distance}};
+    if (distance_bias && last_distance < 0) return fail(MLB_INVALID_ARGUMENT, "attention_tc: a distance bias has a last distance");
     static bool configured_on[MAX_DEVICES] = {false};         // the attribute belongs to the device
     bool& configured = configured_on[device_index()];
     if (!configured) {

@@ -92,6 +92,19 @@ __device__ __forceinline__ int first_visible_key(int pos, int window, int chunk)
     return lo;
 }
 
+// A score bias that depends on the distance query - key and on the head: one row a head, the values of distances 0, 1, ..
+// last with DISTANCE_PAD copies of the first value in front and DISTANCE_PAD copies of the last one behind (every distance
+// beyond `last` has the last one's value), so that a tile's distances around a row's end need no bounds of their own.
+constexpr int DISTANCE_PAD = 256;
+struct DistanceBias {
+    const float* table;        // [heads][DISTANCE_PAD + last + 1 + DISTANCE_PAD], null: none
+    int last;
+    __host__ __device__ __forceinline__ int pitch() const { return last + 1 + 2 * DISTANCE_PAD; }
+    // the row of a head, placed so that row[n] is the bias of distance n
+    __device__ __forceinline__ const float* row(int head) const { return table + (size_t)head * pitch() + DISTANCE_PAD; }
+    __device__ __forceinline__ float at(const float* row, int n) const { return row[min(max(n, 0), last)]; }
+};
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

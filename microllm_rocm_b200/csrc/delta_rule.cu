@@ -14,6 +14,10 @@
 // The scan kernel also runs the two simpler recurrences with a decay per key channel (mlb_linear_scan, `rule`):
 //   rule 1, decayed sum:   S <- diag(g_t) S + k_t v_t^T;   o_t = S^T q_t
 //   rule 2, bonus read:    o_t = (S + diag(u) k_t v_t^T)^T q_t;   then S <- diag(g_t) S + k_t v_t^T      (u [H, DK], fixed)
+// and one with a decay per head (mlb_head_scan):
+//   rule 3, head decay:    S <- g_t S + w_t k_t v_t^T;   o_t = S^T q_t, with one number g per token and head (or one per head,
+//                          fixed) and an optional weight w per token and head.  Optionally a vector n [DK] beside S runs the
+//                          same recurrence with 1 in the place of v: one more column, whose read-out n . q goes to `den`.
 //
 // The order of every addition depends on the token's place in its sequence only, never on how the sequence was cut
 // into steps: a token's result is the same bits however it is scheduled.
@@ -107,7 +111,7 @@ __global__ void __launch_bounds__(WARPS * 32) delta_prepare_kernel(PrepareParams
 struct ScanParams {
     const float* qn; const float* kn;        // [T, G * DK]
     const float* g;                          // [T, H * DK]
-    const float* beta;                       // [T, H] (the delta rule only; else unused and may be null)
+    const float* beta;                       // [T, H]: beta of the delta rule, w of rule 3 (null: 1); else unused and may be null
     const float* bonus;                      // [H, DK] (rule 2 only)
     const float* v; long long ld_v;          // [T, H * DV] (a column block of the convolved rows)
     float* o;                                // [T, H * DV]
@@ -115,6 +119,9 @@ struct ScanParams {
     const int* slots; int num_slots;
     const int* seq_starts; const int* seq_pos0;
     int A, H, G, DK, DV;
+    int g_pitch;                             // rule 3: numbers between two tokens' decays (H; 0: one per head, fixed)
+    float* n_state;                          // rule 3: [slots + 1, H, DK], the vector beside S; null: none
+    float* den;                              // rule 3: [T, H], n . q; given exactly when n_state is
     int vec;                                 // 1: every staged row starts on 16 bytes and is a multiple of four floats long
     int* error_flag;
 };
@@ -140,22 +147,25 @@ __device__ __forceinline__ void copy_async_f32x4(float* to_shared, const float* 
 // CHUNK: tokens whose q, k, g, v and beta are staged in shared memory at a time; the next chunk is copied there
 // asynchronously (cp.async, zero fill for padding) while the present one is computed, so the recurrence never waits for
 // global memory inside a chunk.
-constexpr int RULE_DELTA = 0, RULE_DECAYED_SUM = 1, RULE_BONUS_READ = 2;
+constexpr int RULE_DELTA = 0, RULE_DECAYED_SUM = 1, RULE_BONUS_READ = 2, RULE_HEAD_DECAY = 3;
 
 template <int LANES, int ROWS, int CHUNK, int RULE, int COLS = SCAN_COLS>
 __global__ void __launch_bounds__(COLS * LANES) delta_scan_kernel(ScanParams p) {
     pdl_prologue();
     constexpr int SCAN_LANES = LANES, SCAN_THREADS = COLS * LANES;
     constexpr int DKP = SCAN_LANES * ROWS;                    // padded key width
-    constexpr int PER_TOKEN = 3 * DKP + COLS + 4;        // q | k | g | v of this CTA's columns | beta and three unused
+    constexpr int V_AT = (RULE == RULE_HEAD_DECAY ? 2 : 3) * DKP;
+    constexpr int PER_TOKEN = V_AT + COLS + 4;           // q | k | g (not rule 3) | v of this CTA's columns | beta (rule 3: g, w) and unused
     constexpr int STAGED = CHUNK * PER_TOKEN;
     __shared__ __align__(16) float stage_s[2][STAGED];
-    const int col_blocks = (p.DV + COLS - 1) / COLS;
+    const int all_cols = RULE == RULE_HEAD_DECAY && p.n_state ? p.DV + 1 : p.DV;      // rule 3: the vector beside S is column DV
+    const int col_blocks = (all_cols + COLS - 1) / COLS;
     const int cb = blockIdx.x % col_blocks, h = (blockIdx.x / col_blocks) % p.H, a = blockIdx.x / (col_blocks * p.H);
     const int part = threadIdx.x & (SCAN_LANES - 1);
     const int local_col = threadIdx.x / SCAN_LANES;
     const int col = cb * COLS + local_col;
-    const bool col_ok = col < p.DV;
+    const bool col_ok = col < all_cols;
+    const bool is_n = RULE == RULE_HEAD_DECAY && col == p.DV;                          // (with col_ok only when there is a vector)
     const int start = p.seq_starts[a], n = p.seq_starts[a + 1] - start;
     const int slot = p.slots[a];
     if (slot < 0 || slot >= p.num_slots) {
@@ -165,11 +175,13 @@ __global__ void __launch_bounds__(COLS * LANES) delta_scan_kernel(ScanParams p) 
     const int kvh = h / (p.H / p.G);
     auto row_of = [&](int i) { return (i >> 2) * (4 * LANES) + part * 4 + (i & 3); };
     float S[ROWS];
-    float* st = p.state + (((size_t)slot * p.H + h) * p.DK) * p.DV;
+    // this thread's column of the state, and the distance between its rows
+    float* const st = is_n && col_ok ? p.n_state + ((size_t)slot * p.H + h) * p.DK : p.state + (((size_t)slot * p.H + h) * p.DK) * p.DV + col;
+    const size_t st_pitch = is_n ? 1 : (size_t)p.DV;
     const bool fresh = p.seq_pos0[a] == 0;
 #pragma unroll
     for (int i = 0; i < ROWS; ++i)
-        S[i] = (!fresh && col_ok && row_of(i) < p.DK) ? st[(size_t)row_of(i) * p.DV + col] : 0.0f;
+        S[i] = (!fresh && col_ok && row_of(i) < p.DK) ? st[(size_t)row_of(i) * st_pitch] : 0.0f;
     float U[RULE == RULE_BONUS_READ ? ROWS : 1];
     if (RULE == RULE_BONUS_READ) {
 #pragma unroll
@@ -178,7 +190,7 @@ __global__ void __launch_bounds__(COLS * LANES) delta_scan_kernel(ScanParams p) 
 
     const float* const q_base = p.qn + ((size_t)start * p.G + kvh) * p.DK;
     const float* const k_base = p.kn + ((size_t)start * p.G + kvh) * p.DK;
-    const float* const g_base = p.g + ((size_t)start * p.H + h) * p.DK;
+    const float* const g_base = RULE == RULE_HEAD_DECAY ? p.g + (size_t)start * p.g_pitch + h : p.g + ((size_t)start * p.H + h) * p.DK;
     const float* const v_base = p.v + (size_t)start * p.ld_v + (size_t)h * p.DV;
     const float* const b_base = p.beta ? p.beta + (size_t)start * p.H + h : g_base;     // without beta: any readable address, the value is unused
     const size_t qk_pitch = (size_t)p.G * p.DK, g_pitch = (size_t)p.H * p.DK;
@@ -186,23 +198,26 @@ __global__ void __launch_bounds__(COLS * LANES) delta_scan_kernel(ScanParams p) 
     // tokens beyond the sequence's) becomes zero: a zero k and q keep such rows of S at zero whatever g is
     auto stage = [&](int first, int buf) {
         if (p.vec) {                             // every row a multiple of four floats and 16-byte aligned: four at a time
-            constexpr int UNITS = 3 * DKP / 4 + COLS / 4 + 1;
+            constexpr int UNITS = V_AT / 4 + COLS / 4 + 1;
             for (int e = threadIdx.x; e < CHUNK * UNITS; e += SCAN_THREADS) {
                 const int tok = e / UNITS, u = e % UNITS;
                 const bool live = first + tok < n;
                 const size_t t = live ? (size_t)(first + tok) : 0;
                 float* to = &stage_s[buf][tok * PER_TOKEN];
-                if (u < 3 * DKP / 4) {
+                if (u < V_AT / 4) {
                     const int which = u / (DKP / 4), c = (u % (DKP / 4)) * 4;
                     const bool real = c < p.DK;
                     const float* at = (which == 0 ? q_base + t * qk_pitch : (which == 1 ? k_base + t * qk_pitch : g_base + t * g_pitch)) + (real ? c : 0);
                     copy_async_f32x4(to + which * DKP + c, at, live && real);
                 } else if (u < UNITS - 1) {
-                    const int c = (u - 3 * DKP / 4) * 4, vc = cb * COLS + c;
+                    const int c = (u - V_AT / 4) * 4, vc = cb * COLS + c;
                     const bool real = vc < p.DV;
-                    copy_async_f32x4(to + 3 * DKP + c, v_base + t * p.ld_v + (real ? vc : 0), live && real);
+                    copy_async_f32x4(to + V_AT + c, v_base + t * p.ld_v + (real ? vc : 0), live && real);
+                } else if (RULE == RULE_HEAD_DECAY) {
+                    copy_async_f32(to + V_AT + COLS, g_base + t * p.g_pitch, live);
+                    if (p.beta) copy_async_f32(to + V_AT + COLS + 1, b_base + t * p.H, live);
                 } else {
-                    copy_async_f32(to + 3 * DKP + COLS, b_base + t * p.H, live);
+                    copy_async_f32(to + V_AT + COLS, b_base + t * p.H, live);
                 }
             }
             asm volatile("cp.async.commit_group;" ::: "memory");
@@ -213,14 +228,17 @@ __global__ void __launch_bounds__(COLS * LANES) delta_scan_kernel(ScanParams p) 
             const bool live = first + tok < n;
             const size_t t = live ? (size_t)(first + tok) : 0;
             const int which = w / DKP, c = w % DKP;
-            const int vc = cb * COLS + (w - 3 * DKP);
+            const int vc = cb * COLS + (w - V_AT);
             const float* at;
             bool real;
             if (which == 0) { real = c < p.DK; at = q_base + t * qk_pitch + (real ? c : 0); }
             else if (which == 1) { real = c < p.DK; at = k_base + t * qk_pitch + (real ? c : 0); }
-            else if (which == 2) { real = c < p.DK; at = g_base + t * g_pitch + (real ? c : 0); }
-            else if (w < 3 * DKP + COLS) { real = vc < p.DV; at = v_base + t * p.ld_v + (real ? vc : 0); }
-            else { real = w == 3 * DKP + COLS; at = b_base + t * p.H; }
+            else if (RULE != RULE_HEAD_DECAY && which == 2) { real = c < p.DK; at = g_base + t * g_pitch + (real ? c : 0); }
+            else if (w < V_AT + COLS) { real = vc < p.DV; at = v_base + t * p.ld_v + (real ? vc : 0); }
+            else if (RULE == RULE_HEAD_DECAY) {
+                real = w == V_AT + COLS || (w == V_AT + COLS + 1 && p.beta);
+                at = w == V_AT + COLS + 1 && p.beta ? b_base + t * p.H : g_base + t * p.g_pitch;
+            } else { real = w == V_AT + COLS; at = b_base + t * p.H; }
             copy_async_f32(&stage_s[buf][e], at, live && real);
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
@@ -231,15 +249,22 @@ __global__ void __launch_bounds__(COLS * LANES) delta_scan_kernel(ScanParams p) 
     for (int first = 0, buf = 0; first < n; first += CHUNK, buf ^= 1) {
         if (first + CHUNK < n) stage(first + CHUNK, buf ^ 1);
         const int count = min(CHUNK, n - first);
-        float* const o_at = p.o + ((size_t)start + first) * ((size_t)p.H * p.DV) + (size_t)h * p.DV + col;
+        const size_t o_pitch = is_n ? (size_t)p.H : (size_t)p.H * p.DV;
+        float* const o_at = is_n ? p.den + ((size_t)start + first) * p.H + h
+                                 : p.o + ((size_t)start + first) * ((size_t)p.H * p.DV) + (size_t)h * p.DV + col;
         // `lone`: the lanes of a column meet for this token alone and its o is stored; else the lane's share of o is handed
         // back and the lanes meet once for a group of tokens (below)
         auto token = [&](int tok, bool lone) -> float {
             const float* row = stage_s[buf] + tok * PER_TOKEN;
             const float4* qs = reinterpret_cast<const float4*>(row) + part;
             const float4* ks = reinterpret_cast<const float4*>(row + DKP) + part;
-            const float4* gs = reinterpret_cast<const float4*>(row + 2 * DKP) + part;
-            const float v = row[3 * DKP + local_col], beta = row[3 * DKP + COLS];
+            const float4* gs = reinterpret_cast<const float4*>(row + 2 * DKP) + part;          // (not rule 3)
+            float v = row[V_AT + local_col];
+            const float beta = row[V_AT + COLS];                                               // (rule 3: the head's decay)
+            if (RULE == RULE_HEAD_DECAY) {
+                if (is_n) v = 1.0f;
+                if (p.beta) v *= row[V_AT + COLS + 1];
+            }
             float4 kk[ROWS / 4];
             if (RULE != RULE_DELTA) {
                 // S <- diag(g) S + k v^T with the read-out S^T q behind it (decayed sum), or in front of it with the
@@ -247,7 +272,7 @@ __global__ void __launch_bounds__(COLS * LANES) delta_scan_kernel(ScanParams p) 
                 float o0 = 0.0f, o1 = 0.0f, o2 = 0.0f, o3 = 0.0f;
 #pragma unroll
                 for (int j = 0; j < ROWS / 4; ++j) {
-                    const float4 gg = gs[j * LANES], qq = qs[j * LANES];
+                    const float4 gg = RULE == RULE_HEAD_DECAY ? make_float4(beta, beta, beta, beta) : gs[j * LANES], qq = qs[j * LANES];
                     kk[j] = ks[j * LANES];
                     const float kv0 = kk[j].x * v, kv1 = kk[j].y * v, kv2 = kk[j].z * v, kv3 = kk[j].w * v;
                     if (RULE == RULE_BONUS_READ) {
@@ -256,7 +281,7 @@ __global__ void __launch_bounds__(COLS * LANES) delta_scan_kernel(ScanParams p) 
                     }
                     S[4 * j + 0] = fmaf(S[4 * j + 0], gg.x, kv0); S[4 * j + 1] = fmaf(S[4 * j + 1], gg.y, kv1);
                     S[4 * j + 2] = fmaf(S[4 * j + 2], gg.z, kv2); S[4 * j + 3] = fmaf(S[4 * j + 3], gg.w, kv3);
-                    if (RULE == RULE_DECAYED_SUM) {
+                    if (RULE == RULE_DECAYED_SUM || RULE == RULE_HEAD_DECAY) {
                         o0 = fmaf(S[4 * j + 0], qq.x, o0); o1 = fmaf(S[4 * j + 1], qq.y, o1);
                         o2 = fmaf(S[4 * j + 2], qq.z, o2); o3 = fmaf(S[4 * j + 3], qq.w, o3);
                     }
@@ -265,7 +290,7 @@ __global__ void __launch_bounds__(COLS * LANES) delta_scan_kernel(ScanParams p) 
                 if (!lone) return out;
 #pragma unroll
                 for (int off = LANES / 2; off >= 1; off >>= 1) out += __shfl_xor_sync(0xffffffffu, out, off);
-                if (part == 0 && col_ok) o_at[(size_t)tok * ((size_t)p.H * p.DV)] = out;
+                if (part == 0 && col_ok) o_at[(size_t)tok * o_pitch] = out;
                 return 0.0f;
             }
             float d0 = 0.0f, d1 = 0.0f, d2 = 0.0f, d3 = 0.0f;          // four chains instead of one (always the same four)
@@ -297,7 +322,7 @@ __global__ void __launch_bounds__(COLS * LANES) delta_scan_kernel(ScanParams p) 
             out += __shfl_xor_sync(0xffffffffu, out, 2);
             out += __shfl_xor_sync(0xffffffffu, out, 4);
             if (LANES == 16) out += __shfl_xor_sync(0xffffffffu, out, 8);
-            if (part == 0 && col_ok) o_at[(size_t)tok * ((size_t)p.H * p.DV)] = out;
+            if (part == 0 && col_ok) o_at[(size_t)tok * o_pitch] = out;
             return 0.0f;
         };
         if (count == CHUNK && RULE != RULE_DELTA) {
@@ -328,7 +353,7 @@ __global__ void __launch_bounds__(COLS * LANES) delta_scan_kernel(ScanParams p) 
                         share[i] = keep + __shfl_xor_sync(0xffffffffu, send, off);
                     }
                 }
-                if (part < GROUP && col_ok) o_at[(size_t)(g0 + part) * ((size_t)p.H * p.DV)] = share[0];
+                if (part < GROUP && col_ok) o_at[(size_t)(g0 + part) * o_pitch] = share[0];
             }
         } else if (count == CHUNK) {     // a whole chunk: unrolled, so that a token's read-out runs beside the next token's update
 #pragma unroll
@@ -341,7 +366,7 @@ __global__ void __launch_bounds__(COLS * LANES) delta_scan_kernel(ScanParams p) 
     }
 #pragma unroll
     for (int i = 0; i < ROWS; ++i)
-        if (col_ok && row_of(i) < p.DK) st[(size_t)row_of(i) * p.DV + col] = S[i];
+        if (col_ok && row_of(i) < p.DK) st[(size_t)row_of(i) * st_pitch] = S[i];
 }
 
 // ------------------------------------------------------------------------------ output norm and gate
@@ -433,21 +458,23 @@ namespace {
 template <int RULE>
 int launch_scan(const float* qn, const float* kn, const float* g, const float* beta, const float* bonus, const float* v, long long ld_v,
                 float* o, float* state, const int* slots, int num_slots, const int* seq_starts, const int* seq_pos0,
-                int A, int H, int G, int DK, int DV, int* error_flag, cudaStream_t stream) {
+                int A, int H, int G, int DK, int DV, int* error_flag, cudaStream_t stream, int g_pitch = 0, float* n_state = nullptr,
+                float* den = nullptr) {
     if (A < 0 || H <= 0 || G <= 0 || H % G || DK <= 0 || DK > MAX_D || DV <= 0)
         return fail(MLB_UNSUPPORTED_SIZE, "scan: heads %d/%d, widths %d (at most %d) / %d", H, G, DK, MAX_D, DV);
     if (!qn || !kn || !g || (RULE == RULE_DELTA && !beta) || (RULE == RULE_BONUS_READ && !bonus) || !v || !o || !state || !slots ||
         !seq_starts || !seq_pos0)
         return fail(MLB_INVALID_ARGUMENT, "scan: null operand");
     if (A == 0) return MLB_OK;
-    const bool aligned = ((uintptr_t)qn | (uintptr_t)kn | (uintptr_t)g | (uintptr_t)v) % 16 == 0;
+    const bool aligned = ((uintptr_t)qn | (uintptr_t)kn | (RULE == RULE_HEAD_DECAY ? 0 : (uintptr_t)g) | (uintptr_t)v) % 16 == 0;
     const int vec = aligned && DK % 4 == 0 && DV % 4 == 0 && ld_v % 4 == 0;
-    ScanParams p{qn, kn, g, beta, bonus, v, ld_v, o, state, slots, num_slots, seq_starts, seq_pos0, A, H, G, DK, DV, vec, error_flag};
+    ScanParams p{qn, kn, g, beta, bonus, v, ld_v, o, state, slots, num_slots, seq_starts, seq_pos0, A, H, G, DK, DV,
+                 g_pitch, n_state, den, vec, error_flag};
     // A handful of long-running CTAs (a prompt portion: one CTA walks all its tokens) must be spread one to an SM.  Started
     // early behind a predecessor that still fills the SMs, they land wherever a slot falls free, several on one SM, and
     // the slowest SM decides: such a launch waits for its predecessor the plain way.  Many short CTAs (decoding) start early.
     auto go = [&](auto kernel, int lanes, int cols) {
-        const unsigned blocks = (unsigned)((long long)A * H * ((DV + cols - 1) / cols));
+        const unsigned blocks = (unsigned)((long long)A * H * ((DV + (n_state ? 1 : 0) + cols - 1) / cols));
         const bool early = blocks > 2u * (unsigned)sm_count();
         if (early) launch_kernel(kernel, blocks, cols * lanes, 0, stream, p);
         else kernel<<<blocks, cols * lanes, 0, stream>>>(p);
@@ -480,6 +507,16 @@ MLB_EXPORT int mlb_linear_scan(int rule, const float* q, const float* k, const f
         return launch_scan<RULE_BONUS_READ>(q, k, g, nullptr, bonus, v, ld_v, o, state, slots, num_slots, seq_starts, seq_pos0, A, H, G,
                                             DK, DV, error_flag, stream);
     return fail(MLB_INVALID_ARGUMENT, "linear_scan: unknown rule %d", rule);
+}
+
+// rule 3: S <- g S + w k v^T, o = S^T q.  g [T, H] (per_token 1) or [H] (0, fixed); w [T, H] or null (1).  n_state [slots, H, DK] and
+// den [T, H] together: n <- g n + w k, den = n . q.
+MLB_EXPORT int mlb_head_scan(const float* q, const float* k, const float* g, int per_token, const float* w, const float* v, long long ld_v,
+                             float* o, float* state, float* n_state, float* den, const int* slots, int num_slots, const int* seq_starts,
+                             const int* seq_pos0, int A, int H, int DK, int DV, int* error_flag, cudaStream_t stream) {
+    if ((n_state == nullptr) != (den == nullptr)) return fail(MLB_INVALID_ARGUMENT, "head_scan: the vector's state and its read-out come together");
+    return launch_scan<RULE_HEAD_DECAY>(q, k, g, w, nullptr, v, ld_v, o, state, slots, num_slots, seq_starts, seq_pos0, A, H, H, DK, DV, error_flag,
+                                        stream, per_token ? H : 0, n_state, den);
 }
 
 MLB_EXPORT int mlb_delta_output(const float* o, const float* weight, const float* proj, long long ld_proj, int n_partials,

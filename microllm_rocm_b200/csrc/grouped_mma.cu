@@ -9,7 +9,7 @@
 // bytes, which keeps the eight rows of an ldmatrix phase in different banks.
 // Epilogues: none; times a factor read at the output's own place (fp32); or DUAL: the weight holds two row blocks
 // (gate rows, then `dual_rows` further down the up rows), both are multiplied in the same pass and the result is
-// silu(gate) * up.
+// silu(gate) * up (or the clamped form, gated_value).
 // Sizes must suit 16-byte pieces (K, the row pitches and the column blocks multiples of 8 elements); the caller
 // sends everything else to the CUDA-core kernel.
 #include "common.cuh"
@@ -34,6 +34,7 @@ struct MmaParams {
     const float* factor; long long ldf;
     long long dual_rows;                       // DUAL: the second row block starts this many rows further down
     int M, N, K, G;
+    int act;                                   // DUAL: the activation (gated_value)
 };
 
 __device__ __forceinline__ void cp_async16(void* dst, const void* src, bool valid) {
@@ -53,7 +54,16 @@ __device__ __forceinline__ void mma_bf16(float (&c)[4], const unsigned (&a)[4], 
     asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
                  : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
-__device__ __forceinline__ float silu(float g) { return g / (1.0f + expf(-g)); }
+// act 0: silu(g) * u; larger values are the bits of the clamped form's limit L: g = min(g, L), u = clamp(u, -L, L), g sigmoid(1.702 g) (u + 1)
+__device__ __forceinline__ float gated_value(float g, float u, int act) {
+    if (act > 1) {
+        const float limit = __int_as_float(act);
+        g = fminf(g, limit);
+        u = fminf(fmaxf(u, -limit), limit);
+        return g * (1.0f / (1.0f + expf(-1.702f * g))) * (u + 1.0f);
+    }
+    return g / (1.0f + expf(-g)) * u;
+}
 
 __host__ __device__ constexpr int threads_of(int bm) { return bm == 128 ? 256 : 128; }
 constexpr size_t smem_of(int bm, bool dual) {
@@ -229,7 +239,7 @@ grouped_mma_kernel(MmaParams p) {
                 if (n >= p.N) continue;
                 const size_t col = (size_t)group * p.c_group_cols + n;
                 float v = acc[m][0][j][half * 2 + i];
-                if (DUAL) v = silu(v) * acc[m][NB - 1][j][half * 2 + i];
+                if (DUAL) v = gated_value(v, acc[m][NB - 1][j][half * 2 + i], p.act);
                 if (p.factor) v *= p.factor[(size_t)c * p.ldf + col];
                 ((OutT*)p.C)[(size_t)c * p.ldc + col] = from_f32<OutT>(v);
             }
@@ -257,20 +267,22 @@ void launch(const MmaParams& p, int row_tile, unsigned tiles_y, cudaStream_t str
 
 }  // namespace
 
-// dual_rows > 0: W holds gate rows [0, N) and up rows [dual_rows, dual_rows + N) per group; C = silu(A gate^T) * (A up^T).
+// dual_rows > 0: W holds gate rows [0, N) and up rows [dual_rows, dual_rows + N) per group; C = silu(A gate^T) * (A up^T), or the
+// clamped form when `act` holds the bits of its limit.
 MLB_EXPORT int mlb_grouped_mma(const void* A, long long lda, long long a_group_cols, const void* W, long long ldw,
                                long long w_group_stride, void* C, long long ldc, long long c_group_cols,
                                const int* group_offsets, const int* a_rows, const int* c_rows, int a_row_div,
                                const float* factor, long long ldf, long long dual_rows, int M, int N, int K, int G,
-                               int out_dtype, int row_tile, cudaStream_t stream) {
+                               int out_dtype, int row_tile, int act, cudaStream_t stream) {
     if (M < 0 || N <= 0 || K <= 0 || G <= 0 || a_row_div <= 0 || dual_rows < 0 || (row_tile != 16 && row_tile != 64 && row_tile != 128))
         return fail(MLB_INVALID_ARGUMENT, "grouped_mma: bad sizes M=%d N=%d K=%d G=%d", M, N, K, G);
     if (K % 8 || lda % 8 || ldw % 8 || a_group_cols % 8 || w_group_stride % 8 || (uintptr_t)A % 16 || (uintptr_t)W % 16)
         return fail(MLB_UNSUPPORTED_SIZE, "grouped_mma: K, the row pitches and the column blocks must be multiples of 8 elements");
+    if (act < 0 || act == 1) return fail(MLB_INVALID_ARGUMENT, "grouped_mma: unknown activation %d", act);
     if (group_offsets && G > MAX_GROUPS) return fail(MLB_UNSUPPORTED_SIZE, "grouped_mma: more than %d groups", MAX_GROUPS);
     if (M == 0) return MLB_OK;
     MmaParams p{(const __nv_bfloat16*)A, lda, a_group_cols, (const __nv_bfloat16*)W, ldw, w_group_stride, C, ldc, c_group_cols,
-                group_offsets, a_rows, c_rows, a_row_div, factor, ldf, dual_rows, M, N, K, G};
+                group_offsets, a_rows, c_rows, a_row_div, factor, ldf, dual_rows, M, N, K, G, act};
     const long long per = (M + row_tile - 1) / row_tile;
     const long long tiles = group_offsets ? per + G : per * G;
     if (tiles > 65535) return fail(MLB_UNSUPPORTED_SIZE, "grouped_mma: %lld row tiles exceed one launch", tiles);

@@ -1,4 +1,4 @@
-// Layer norm with weight and bias, fp32:  y = (v - mean(v)) / sqrt(mean((v - mean)^2) + eps) * w + b.
+// Layer norm with weight and (optional: null) bias, fp32:  y = (v - mean(v)) / sqrt(mean((v - mean)^2) + eps) * w + b.
 //
 //   mlb_layernorm             y[r] = LN(x[rows[r]] or x[r]), stored in the compute dtype (the final norm on selected rows)
 //   mlb_scale_add_layernorm   x[r] <- LN(alpha * x[r] + s1 * sum_k d1[k][r] + s2 * sum_k d2[k][r]) in place (the stream of a
@@ -61,7 +61,10 @@ __global__ void __launch_bounds__(LN_THREADS) layernorm_kernel(LnParams p) {
 #pragma unroll
             for (int i = 0; i < LN_VECS; ++i) {
                 const int c = (threadIdx.x + i * LN_THREADS) * 4;
-                if (c < W) { wv[i] = *reinterpret_cast<const float4*>(p.weight + c); bv[i] = *reinterpret_cast<const float4*>(p.bias + c); }
+                if (c < W) {
+                    wv[i] = *reinterpret_cast<const float4*>(p.weight + c);
+                    bv[i] = p.bias ? *reinterpret_cast<const float4*>(p.bias + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+                }
             }
         }
         pdl_wait();
@@ -98,7 +101,7 @@ __global__ void __launch_bounds__(LN_THREADS) layernorm_kernel(LnParams p) {
             const int c = (threadIdx.x + i * LN_THREADS) * 4;
             if (c >= W) break;
             const float4 w4 = FEW ? wv[FEW ? i : 0] : *reinterpret_cast<const float4*>(p.weight + c);
-            const float4 b4 = FEW ? bv[FEW ? i : 0] : *reinterpret_cast<const float4*>(p.bias + c);
+            const float4 b4 = FEW ? bv[FEW ? i : 0] : (p.bias ? *reinterpret_cast<const float4*>(p.bias + c) : make_float4(0.f, 0.f, 0.f, 0.f));
             float4 y;
             y.x = v[i].x * inv * w4.x + b4.x; y.y = v[i].y * inv * w4.y + b4.y;
             y.z = v[i].z * inv * w4.z + b4.z; y.w = v[i].w * inv * w4.w + b4.w;
@@ -149,7 +152,7 @@ __global__ void __launch_bounds__(LN_THREADS) layernorm_kernel(LnParams p) {
     const float inv = 1.0f / sqrtf(block_sum(sq, scratch) / (float)W + p.eps);
     OutT* yr = p.out ? (OutT*)p.out + (size_t)r * W : nullptr;
     for (int c = threadIdx.x; c < W; c += LN_THREADS) {
-        const float y = (row_s[c] - mean) * inv * p.weight[c] + p.bias[c];
+        const float y = (row_s[c] - mean) * inv * p.weight[c] + (p.bias ? p.bias[c] : 0.0f);
         if (ADD) xr[c] = y;
         if (yr) yr[c] = from_f32<OutT>(y);
     }
@@ -183,7 +186,7 @@ int launch(const LnParams& p, int n, int out_dtype, bool add, cudaStream_t strea
 
 MLB_EXPORT int mlb_layernorm(const float* x, const float* weight, const float* bias, void* out, int out_dtype, const int* rows,
                              int n, int width, float eps, cudaStream_t stream) {
-    if (!x || !weight || !bias || !out) return fail(MLB_INVALID_ARGUMENT, "layernorm: null operand");
+    if (!x || !weight || !out) return fail(MLB_INVALID_ARGUMENT, "layernorm: null operand");
     LnParams p{};
     p.x = const_cast<float*>(x); p.weight = weight; p.bias = bias; p.out = out; p.rows = rows; p.width = width; p.eps = eps;
     return launch(p, n, out_dtype, false, stream, "layernorm");
@@ -192,7 +195,7 @@ MLB_EXPORT int mlb_layernorm(const float* x, const float* weight, const float* b
 MLB_EXPORT int mlb_scale_add_layernorm(float* x, float alpha, const float* d1, int n1, long long stride1, float s1, const float* d2,
                                        int n2, long long stride2, float s2, const float* weight, const float* bias, void* out,
                                        int out_dtype, int n, int width, float eps, cudaStream_t stream) {
-    if (!x || !d1 || !weight || !bias || n1 < 1 || (d2 && n2 < 1)) return fail(MLB_INVALID_ARGUMENT, "scale_add_layernorm: bad operands");
+    if (!x || !d1 || !weight || n1 < 1 || (d2 && n2 < 1)) return fail(MLB_INVALID_ARGUMENT, "scale_add_layernorm: bad operands");
     LnParams p{};
     p.x = x; p.d1 = d1; p.n1 = n1; p.stride1 = stride1; p.s1 = s1; p.d2 = d2; p.n2 = n2; p.stride2 = stride2; p.s2 = s2;
     p.alpha = alpha; p.weight = weight; p.bias = bias; p.out = out; p.width = width; p.eps = eps;

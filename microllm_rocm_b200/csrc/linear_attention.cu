@@ -14,6 +14,13 @@
 //                          times act(gate) with the gate read from a projection's fp32 output (sigmoid or silu).
 //   mlb_lightning_prepare  what enters a recurrence with ONE fixed decay per head: q, k, v = silu of their projection columns
 //                          (fp32, partial results summed in split order) and the head's decay written for each of its key channels.
+//   mlb_head_decay_prepare what enters a recurrence with one decay per head: q * q_scale, k * k_scale and v gathered out of a
+//                          projection's fp32 output, q and k turned on the first rot_dims elements of every head (element i with
+//                          i + rot_dims / 2; sines and cosines from a table of the step), the scales behind the rotation.  In the
+//                          same launch, optionally, the gates of a matrix memory with exponential gates: per token and head
+//                          i = c tanh((a + b_i) / c), f = log_sigmoid(c tanh((a' + b_f) / c)), m_t = max(f + m_(t-1), i) from the
+//                          sequence's state (0 at position 0) and back into it; keep = exp(f + m_(t-1) - m_t), take = exp(i - m_t),
+//                          floor = exp(-m_t).  The walk over m is serial in the token, the same operations however it is cut.
 //   mlb_row_norm_gate      o / sqrt(mean(o^2) + eps) over the WHOLE row (all heads together), times a weight of the row's length,
 //                          times sigmoid(gate) element by element.
 #include "common.cuh"
@@ -249,8 +256,13 @@ struct OutputParams {
     const float* o;                          // [T, H * DV]
     const float* weight; int weight_per_head;      // [DV] shared by the heads (0) or [H * DV] (1); null: no weight
     Columns gate; int gate_col; int gate_act;      // gate.base null: no gate; 0 sigmoid, 1 silu
+    const float* den; const float* floor;    // [T, H], both or none: o is first divided by max(|den|, floor) + den_eps
+    float den_eps;
     void* out;                               // [T, H * DV]
     int T, H, DV; float eps;
+    __device__ __forceinline__ float divisor(int t, int h) const {
+        return den ? fmaxf(fabsf(den[(size_t)t * H + h]), floor[(size_t)t * H + h]) + den_eps : 1.0f;
+    }
 };
 
 template <typename OutT>
@@ -261,12 +273,14 @@ __global__ void __launch_bounds__(WARPS * 32) head_norm_gate_kernel(OutputParams
     if (item >= (long long)p.T * p.H) return;
     const int t = (int)(item / p.H), h = (int)(item % p.H);
     const float* src = p.o + ((size_t)t * p.H + h) * p.DV;
+    const float by = p.divisor(t, h);
     float x[PER_LANE];
     float ss = 0.0f;
 #pragma unroll
     for (int i = 0; i < PER_LANE; ++i) {
         const int c = lane + 32 * i;
         x[i] = c < p.DV ? src[c] : 0.0f;
+        if (p.den) x[i] /= by;
         ss = fmaf(x[i], x[i], ss);
     }
     const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)p.DV + p.eps);
@@ -295,6 +309,7 @@ __global__ void __launch_bounds__(WARPS * 32) head_norm_gate_x4_kernel(OutputPar
     if (item >= (long long)p.T * p.H) return;
     const int t = (int)(item / p.H), h = (int)(item % p.H);
     const float* src = p.o + ((size_t)t * p.H + h) * p.DV;
+    const float by = p.divisor(t, h);
     float4 x[QUADS], g[QUADS];
     float ss = 0.0f;
 #pragma unroll
@@ -302,6 +317,7 @@ __global__ void __launch_bounds__(WARPS * 32) head_norm_gate_x4_kernel(OutputPar
         const int c = 4 * lane + 128 * i;
         x[i] = c < p.DV ? *reinterpret_cast<const float4*>(src + c) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
         if (p.gate.base && c < p.DV) g[i] = p.gate.at4(t, p.gate_col + h * p.DV + c);
+        if (p.den) { x[i].x /= by; x[i].y /= by; x[i].z /= by; x[i].w /= by; }
         ss = fmaf(x[i].x, x[i].x, ss); ss = fmaf(x[i].y, x[i].y, ss); ss = fmaf(x[i].z, x[i].z, ss); ss = fmaf(x[i].w, x[i].w, ss);
     }
     const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)p.DV + p.eps);
@@ -403,13 +419,14 @@ MLB_EXPORT int mlb_decay_prepare(const float* q, long long q_ld, int q_partials,
 }
 
 MLB_EXPORT int mlb_head_norm_gate(const float* o, const float* weight, int weight_per_head, const float* gate, long long gate_ld,
-                                  int gate_partials, long long gate_stride, int gate_col, int gate_act, void* out, int out_dtype,
-                                  int T, int H, int DV, float eps, cudaStream_t stream) {
+                                  int gate_partials, long long gate_stride, int gate_col, int gate_act, const float* den,
+                                  const float* floor, float den_eps, void* out, int out_dtype, int T, int H, int DV, float eps,
+                                  cudaStream_t stream) {
     if (T < 0 || H <= 0 || DV <= 0 || DV > MAX_D) return fail(MLB_UNSUPPORTED_SIZE, "head_norm_gate: value width %d (at most %d)", DV, MAX_D);
-    if (!o || !out) return fail(MLB_INVALID_ARGUMENT, "head_norm_gate: null operand");
+    if (!o || !out || (den == nullptr) != (floor == nullptr)) return fail(MLB_INVALID_ARGUMENT, "head_norm_gate: null operand");
     if (T == 0) return MLB_OK;
     OutputParams p{o, weight, weight_per_head, Columns{gate, gate_ld, gate_partials < 1 ? 1 : gate_partials, gate_stride}, gate_col,
-                   gate_act, out, T, H, DV, eps};
+                   gate_act, den, floor, den_eps, out, T, H, DV, eps};
     const long long items = (long long)T * H;
     const unsigned blocks = (unsigned)((items + WARPS - 1) / WARPS);
     const bool fours = DV % 4 == 0 && p.gate.fours(gate_col) && ((uintptr_t)o | (uintptr_t)weight | (uintptr_t)out) % 16 == 0;
@@ -522,4 +539,146 @@ MLB_EXPORT int mlb_row_norm_gate(const float* o, const float* weight, const floa
         launch_kernel(row_norm_gate_kernel<float>, (unsigned)T, ROW_THREADS, 0, stream, o, weight, g, gate_col, (float*)out, width, eps);
     else return fail(MLB_INVALID_ARGUMENT, "row_norm_gate: unsupported dtype %d", out_dtype);
     return check_launch("row_norm_gate");
+}
+
+namespace {
+
+constexpr int PREPARE_THREADS = 256;
+
+struct HeadPrepareParams {
+    Columns src; int q_col, k_col, v_col;
+    const float2* cos_sin; int rot_dims;           // [T, rot_dims / 2]; rot_dims 0: no rotation
+    float q_scale, k_scale;
+    float* q_out; float* k_out; float* v_out;      // [T, H * DK] x 2, [T, H * DV]
+    int T, H, DK, DV;
+    // the gates (gate_blocks 0: none)
+    int gate_blocks, i_col, f_col;
+    const float* i_bias; const float* f_bias;      // [H]
+    float cap;
+    float* m_state; const int* slots; int num_slots;        // [slots + 1, H]
+    const int* seq_starts; const int* seq_pos0; int A;
+    float* keep; float* take; float* floor;        // [T, H]
+    int* error_flag;
+};
+
+// One warp walks the tokens of one (sequence, head): the logs of 32 tokens' gates side by side in its lanes, the running
+// maximum from lane to lane, the exponentials side by side again.  The next 32 tokens' columns are fetched meanwhile.
+__device__ __forceinline__ void walk_gates(const HeadPrepareParams& p, int item) {
+    const int lane = threadIdx.x & 31, a = item / p.H, h = item % p.H;
+    const int start = p.seq_starts[a], n = p.seq_starts[a + 1] - start;
+    const int slot = p.slots[a];
+    if (slot < 0 || slot >= p.num_slots) {
+        if (lane == 0 && p.error_flag) atomicExch(p.error_flag, 3);
+        return;
+    }
+    float m = p.seq_pos0[a] == 0 ? 0.0f : p.m_state[(size_t)slot * p.H + h];
+    const float bi = p.i_bias[h], bf = p.f_bias[h];
+    float ai = 0.0f, af = 0.0f;
+    if (lane < n) { ai = p.src.at(start + lane, p.i_col + h); af = p.src.at(start + lane, p.f_col + h); }
+    for (int base = 0; base < n; base += 32) {
+        const float i = p.cap * tanhf((ai + bi) / p.cap);
+        const float f = log_sigmoid(p.cap * tanhf((af + bf) / p.cap));
+        const int next = base + 32 + lane;
+        if (next < n) { ai = p.src.at(start + next, p.i_col + h); af = p.src.at(start + next, p.f_col + h); }
+        const int count = min(32, n - base);
+        float before = 0.0f, now = 0.0f;
+#pragma unroll
+        for (int j = 0; j < 32; ++j) {
+            const float fj = __shfl_sync(0xffffffffu, f, j), ij = __shfl_sync(0xffffffffu, i, j);
+            const float m_new = fmaxf(fj + m, ij);
+            if (lane == j) { before = m; now = m_new; }
+            if (j < count) m = m_new;
+        }
+        if (lane < count) {
+            const size_t at = (size_t)(start + base + lane) * p.H + h;
+            p.keep[at] = expf(f + before - now);
+            p.take[at] = expf(i - now);
+            p.floor[at] = expf(-now);
+        }
+    }
+    if (lane == 0) p.m_state[(size_t)slot * p.H + h] = m;
+}
+
+// what a column of q or k becomes: turned with its partner where it belongs to the turned part of its head, then scaled
+__device__ __forceinline__ float turned(const HeadPrepareParams& p, long long t, int col, int c, float scale) {
+    const int hc = c % p.DK, half = p.rot_dims / 2;
+    const float own = p.src.at(t, col + c);
+    if (hc >= p.rot_dims) return own * scale;
+    const bool first = hc < half;
+    const float other = p.src.at(t, col + (first ? c + half : c - half));
+    const float2 cs = p.cos_sin[t * half + (first ? hc : hc - half)];
+    return (first ? own * cs.x - other * cs.y : own * cs.x + other * cs.y) * scale;
+}
+
+// FOUR: four neighbouring columns a thread (16-byte loads and stores); DK, DV, rot_dims / 2 and the columns are multiples of 4
+template <bool FOUR>
+__global__ void __launch_bounds__(PREPARE_THREADS) head_decay_prepare_kernel(HeadPrepareParams p) {
+    pdl_prologue();
+    if ((int)blockIdx.x < p.gate_blocks) {                  // the serial part first: it takes longest
+        const int item = blockIdx.x * (PREPARE_THREADS / 32) + (threadIdx.x >> 5);
+        if (item < p.A * p.H) walk_gates(p, item);
+        return;
+    }
+    constexpr int N = FOUR ? 4 : 1;
+    const int HK = p.H * p.DK, HV = p.H * p.DV, per = (2 * HK + HV) / N;
+    const long long i = (long long)(blockIdx.x - p.gate_blocks) * PREPARE_THREADS + threadIdx.x;
+    if (i >= p.T * (long long)per) return;
+    const long long t = i / per;
+    int c = (int)(i % per) * N;
+    if (c >= 2 * HK) {
+        c -= 2 * HK;
+        if (FOUR) *reinterpret_cast<float4*>(p.v_out + t * HV + c) = p.src.at4(t, p.v_col + c);
+        else p.v_out[t * HV + c] = p.src.at(t, p.v_col + c);
+        return;
+    }
+    const bool is_q = c < HK;
+    if (!is_q) c -= HK;
+    float* const out = (is_q ? p.q_out : p.k_out) + t * HK + c;
+    const int col = is_q ? p.q_col : p.k_col;
+    const float scale = is_q ? p.q_scale : p.k_scale;
+    if (!FOUR) { *out = turned(p, t, col, c, scale); return; }
+    float4 own = p.src.at4(t, col + c);
+    const int hc = c % p.DK, half = p.rot_dims / 2;
+    if (hc < p.rot_dims) {
+        const bool first = hc < half;
+        const float4 other = p.src.at4(t, col + (first ? c + half : c - half));
+        const float4* cs = reinterpret_cast<const float4*>(p.cos_sin + t * half + (first ? hc : hc - half));
+        const float4 cs0 = cs[0], cs1 = cs[1];              // cos, sin of two pairs each
+        const float sign = first ? -1.0f : 1.0f;
+        own.x = own.x * cs0.x + sign * other.x * cs0.y; own.y = own.y * cs0.z + sign * other.y * cs0.w;
+        own.z = own.z * cs1.x + sign * other.z * cs1.y; own.w = own.w * cs1.z + sign * other.w * cs1.w;
+    }
+    own.x *= scale; own.y *= scale; own.z *= scale; own.w *= scale;
+    *reinterpret_cast<float4*>(out) = own;
+}
+
+}  // namespace
+
+// cos_sin [T, rot_dims / 2] (cos, sin) pairs; i_bias null: no gates (then everything behind k_scale up to A is unused)
+MLB_EXPORT int mlb_head_decay_prepare(const float* src, long long ld, int n_partials, long long partial_stride, int q_col, int k_col,
+                                      int v_col, const float* cos_sin, int rot_dims, float q_scale, float k_scale, float* q_out,
+                                      float* k_out, float* v_out, int T, int H, int DK, int DV, int i_col, int f_col,
+                                      const float* i_bias, const float* f_bias, float cap, float* m_state, const int* slots,
+                                      int num_slots, const int* seq_starts, const int* seq_pos0, int A, float* gates,
+                                      int* error_flag, cudaStream_t stream) {
+    if (T < 0 || A < 0 || H <= 0 || DK <= 0 || DV <= 0 || n_partials < 1 || !src || !q_out || !k_out || !v_out || rot_dims < 0 || rot_dims % 2 ||
+        rot_dims > DK || (rot_dims > 0 && !cos_sin))
+        return fail(MLB_INVALID_ARGUMENT, "head_decay_prepare: bad operands");
+    if (i_bias && (!f_bias || !m_state || !slots || !seq_starts || !seq_pos0 || !gates || !(cap > 0.0f)))
+        return fail(MLB_INVALID_ARGUMENT, "head_decay_prepare: the gates need biases, a cap, a state and the step's sequences");
+    if (T == 0) return MLB_OK;
+    const int warps = PREPARE_THREADS / 32;
+    const size_t plane = (size_t)T * H;
+    HeadPrepareParams p{Columns{src, ld, n_partials, partial_stride}, q_col, k_col, v_col, (const float2*)cos_sin, rot_dims, q_scale, k_scale,
+                        q_out, k_out, v_out, T, H, DK, DV, i_bias ? (A * H + warps - 1) / warps : 0, i_col, f_col, i_bias, f_bias, cap,
+                        m_state, slots, num_slots, seq_starts, seq_pos0, A, gates, gates ? gates + plane : nullptr,
+                        gates ? gates + 2 * plane : nullptr, error_flag};
+    const long long n = (long long)T * (2LL * H * DK + (long long)H * DV);
+    const bool fours = DK % 4 == 0 && DV % 4 == 0 && (rot_dims / 2) % 4 == 0 && p.src.fours(q_col) && p.src.fours(k_col) && p.src.fours(v_col) &&
+                       ((uintptr_t)q_out | (uintptr_t)k_out | (uintptr_t)v_out | (uintptr_t)cos_sin) % 16 == 0;
+    const long long work = fours ? n / 4 : n;
+    const unsigned blocks = (unsigned)(p.gate_blocks + (work + PREPARE_THREADS - 1) / PREPARE_THREADS);
+    if (fours) launch_kernel(head_decay_prepare_kernel<true>, blocks, PREPARE_THREADS, 0, stream, p);
+    else launch_kernel(head_decay_prepare_kernel<false>, blocks, PREPARE_THREADS, 0, stream, p);
+    return check_launch("head_decay_prepare");
 }

@@ -5,6 +5,9 @@
 //                 Optionally one more column (the gate of a shared expert) whose sigmoid is stored per token.
 //                 `scoring` 1: s = softmax(z) over ALL outputs (no bias inside); the `top` largest s[e] + b[e] are chosen
 //                 (b a correction that only steers the choice) and the weights are the chosen s themselves, not renormalised.
+//                 `scoring` 2: s = sigmoid(z); the experts form `groups` equal groups of neighbours, a group scores the sum of its
+//                 two largest s[e] + b[e] and only experts of the `keep` best groups can be chosen; the `top` largest of those
+//                 run with weights s / (sum of the chosen s + 1e-20) * weight_scale.
 //   moe_align     (below) skips, without raising the flag, ids in [experts, experts + passthrough): outputs of the router that
 //                 have no expert behind them (moe_combine adds the token's own input times the weight for those).
 //   moe_align     from ids[T*top] to a list of the pairs (token, choice) sorted by expert: offsets[E+1] and
@@ -29,19 +32,50 @@ constexpr int MAX_TOP = 32;       // one chosen logit per lane
 __global__ void __launch_bounds__(ROUTE_WARPS * 32)
 moe_select_kernel(const float* __restrict__ logits, long long ld, int n_partials, long long partial_stride,
                   const float* __restrict__ bias, int gate_col, int tokens, int experts, int top,
-                  int* __restrict__ ids, float* __restrict__ weights, float* __restrict__ gate_out, int scoring) {
+                  int* __restrict__ ids, float* __restrict__ weights, float* __restrict__ gate_out, int scoring, int groups, int keep,
+                  float weight_scale) {
     pdl_prologue();
-    extern __shared__ float logits_s[];                 // [ROUTE_WARPS][experts] (scoring 1: twice that, choice scores then s)
+    extern __shared__ float logits_s[];                 // [ROUTE_WARPS][experts] (scoring 1: twice that, choice scores then s; 2: and the groups' scores)
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int t = blockIdx.x * ROUTE_WARPS + warp;
     if (t >= tokens) return;
-    float* z = logits_s + (size_t)warp * experts * (scoring == 1 ? 2 : 1);
-    float* score = z + experts;                         // scoring 1 only
+    float* z = logits_s + (size_t)warp * experts * (scoring + 1);
+    float* score = z + experts;                         // scoring 1 and 2 only
     const float* row = logits + (size_t)t * ld;
     for (int e = lane; e < experts; e += 32) {
         float v = row[e];
         for (int k = 1; k < n_partials; ++k) v += row[(size_t)k * partial_stride + e];
-        z[e] = scoring == 1 ? v : v + (bias ? bias[e] : 0.0f);
+        z[e] = scoring >= 1 ? v : v + (bias ? bias[e] : 0.0f);
+    }
+    if (scoring == 2) {
+        for (int e = lane; e < experts; e += 32) {      // (every lane turns its own elements)
+            const float v = z[e], sc = v >= 0.0f ? 1.0f / (1.0f + expf(-v)) : expf(v) / (1.0f + expf(v));
+            score[e] = sc;
+            z[e] = sc + (bias ? bias[e] : 0.0f);
+        }
+        __syncwarp();
+        if (keep < groups) {
+            float* group_score = score + experts;
+            const int size = experts / groups;
+            for (int g = lane; g < groups; g += 32) {
+                float first = -INFINITY, second = -INFINITY;
+                for (int e = g * size; e < (g + 1) * size; ++e) {
+                    const float v = z[e];
+                    if (v > first) { second = first; first = v; }
+                    else if (v > second) second = v;
+                }
+                group_score[g] = size > 1 ? first + second : first;
+            }
+            __syncwarp();
+            // a group is kept when fewer than `keep` groups stand before it (larger score, or the same and a smaller index)
+            for (int e = lane; e < experts; e += 32) {
+                const int own = e / size;
+                const float mine = group_score[own];
+                int before = 0;
+                for (int g = 0; g < groups; ++g) before += group_score[g] > mine || (group_score[g] == mine && g < own);
+                if (before >= keep) z[e] = nanf("");    // never chosen (below)
+            }
+        }
     }
     if (scoring == 1) {
         __syncwarp();
@@ -81,12 +115,17 @@ moe_select_kernel(const float* __restrict__ logits, long long ld, int n_partials
         }
         if (best == 0x7fffffff) { best = 0; best_v = 0.0f; }      // nothing left that is a number
         if (j == 0) first = best_v;
-        if (lane == (j & 31)) chosen = scoring == 1 ? score[best] : best_v;
+        if (lane == (j & 31)) chosen = scoring >= 1 ? score[best] : best_v;
         if (lane == 0) { ids[(size_t)t * top + j] = best; z[best] = nanf(""); }
         __syncwarp();
     }
     if (scoring == 1) {
         if (lane < top) weights[(size_t)t * top + lane] = chosen;
+        return;
+    }
+    if (scoring == 2) {
+        const float total = warp_sum(lane < top ? chosen : 0.0f) + 1e-20f;
+        if (lane < top) weights[(size_t)t * top + lane] = chosen / total * weight_scale;
         return;
     }
     const float w = lane < top ? expf(chosen - first) : 0.0f;
@@ -150,15 +189,18 @@ __global__ void moe_combine_kernel(const float* __restrict__ y, const float* __r
 
 MLB_EXPORT int mlb_moe_select(const float* logits, long long ld, int n_partials, long long partial_stride, const float* bias,
                               int gate_col, int tokens, int experts, int top, int* ids, float* weights, float* gate_out,
-                              int scoring, cudaStream_t stream) {
-    if (scoring != 0 && scoring != 1) return fail(MLB_INVALID_ARGUMENT, "moe_select: unknown scoring %d", scoring);
+                              int scoring, int groups, int keep, float weight_scale, cudaStream_t stream) {
+    if (scoring < 0 || scoring > 2) return fail(MLB_INVALID_ARGUMENT, "moe_select: unknown scoring %d", scoring);
+    if (scoring == 2 && (groups <= 0 || experts % groups || keep <= 0 || keep > groups || top > keep * (experts / groups)))
+        return fail(MLB_INVALID_ARGUMENT, "moe_select: %d of %d groups of %d experts, top %d", keep, groups, experts, top);
     if (tokens < 0 || experts <= 0 || experts > MAX_EXPERTS || top <= 0 || top > experts || top > MAX_TOP || n_partials < 1 ||
         ld < experts || gate_col >= ld)
         return fail(MLB_INVALID_ARGUMENT, "moe_select: bad sizes (experts %d, top %d; at most %d and %d)", experts, top, MAX_EXPERTS, MAX_TOP);
     if (tokens == 0) return MLB_OK;
     const unsigned blocks = (tokens + ROUTE_WARPS - 1) / ROUTE_WARPS;
-    launch_kernel(moe_select_kernel, blocks, ROUTE_WARPS * 32, (size_t)ROUTE_WARPS * experts * sizeof(float) * (scoring == 1 ? 2 : 1),
-                  stream, logits, ld, n_partials, partial_stride, bias, gate_col, tokens, experts, top, ids, weights, gate_out, scoring);
+    launch_kernel(moe_select_kernel, blocks, ROUTE_WARPS * 32, (size_t)ROUTE_WARPS * experts * sizeof(float) * (scoring + 1),
+                  stream, logits, ld, n_partials, partial_stride, bias, gate_col, tokens, experts, top, ids, weights, gate_out, scoring, groups, keep,
+                  weight_scale);
     return check_launch("moe_select");
 }
 

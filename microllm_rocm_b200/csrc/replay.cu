@@ -30,7 +30,7 @@ MLB_DEFINE_LAST_ERROR()
 
 namespace {
 
-constexpr int MAX_INT_SLOTS = 28;
+constexpr int MAX_INT_SLOTS = 32;
 constexpr int MAX_FLOAT_SLOTS = 4;
 
 }  // namespace
@@ -48,6 +48,7 @@ struct MlbCallRecord {
 };
 
 typedef int (*GenericLauncher)(unsigned long long, unsigned long long, unsigned long long, unsigned long long,
+                               unsigned long long, unsigned long long, unsigned long long, unsigned long long,
                                unsigned long long, unsigned long long, unsigned long long, unsigned long long,
                                unsigned long long, unsigned long long, unsigned long long, unsigned long long,
                                unsigned long long, unsigned long long, unsigned long long, unsigned long long,
@@ -86,7 +87,7 @@ MLB_EXPORT int mlb_replay_calls(const MlbCallRecord* records, int count, const u
         const float* f = rec.floats;
         const int status = ((GenericLauncher)rec.function)(
             a[0], a[1], a[2], a[3], a[4], a[5], a[6], a[7], a[8], a[9], a[10], a[11], a[12], a[13], a[14], a[15], a[16],
-            a[17], a[18], a[19], a[20], a[21], a[22], a[23], a[24], a[25], a[26], a[27], f[0], f[1], f[2], f[3]);
+            a[17], a[18], a[19], a[20], a[21], a[22], a[23], a[24], a[25], a[26], a[27], a[28], a[29], a[30], a[31], f[0], f[1], f[2], f[3]);
         ++made;
         if (status != 0) {
             if (failed_at) *failed_at = r;

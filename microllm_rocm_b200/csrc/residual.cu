@@ -1,6 +1,6 @@
 // Residual-stream kernels of decoders whose blocks scale what they add:
 //
-//   embed_gather_scaled   out[t,:] = table[id[t],:] * scale               (bad id -> NaN)
+//   embed_gather_scaled   out[t,:] = table[id[t],:] * scale               (bad id -> NaN), written `copies` times side by side
 //   add_table_rows        x[t,:] += table[index[t],:]                     learned additive positions
 //   add_scaled_rmsnorm    x[t,:] += s[:] * sum_k delta_k[t,:];  out[t,:] = x[t,:] / sqrt(mean(x^2) + eps) * w[:]
 //   add_scaled_inplace    x[t,:] += s[:] * sum_k delta_k[t,:]
@@ -26,18 +26,18 @@ constexpr int ROW_THREADS = 256;
 
 template <typename TableT>
 __global__ void embed_scaled_kernel(const TableT* __restrict__ table, const int* __restrict__ ids, float* __restrict__ out,
-                                    int tokens, int width, int vocab, float scale) {
+                                    int tokens, int width, int vocab, float scale, int copies) {
     pdl_prologue();
     const int t = blockIdx.x;
     if (t >= tokens) return;
     const int id = ids[t];
-    float* dst = out + (size_t)t * width;
-    if (id < 0 || id >= vocab) {
-        for (int c = threadIdx.x; c < width; c += blockDim.x) dst[c] = nanf("");
-        return;
+    const bool known = id >= 0 && id < vocab;
+    float* dst = out + (size_t)t * copies * width;
+    const TableT* src = table + (size_t)(known ? id : 0) * width;
+    for (int c = threadIdx.x; c < width; c += blockDim.x) {
+        const float v = known ? to_f32(src[c]) * scale : nanf("");
+        for (int s = 0; s < copies; ++s) dst[(size_t)s * width + c] = v;
     }
-    const TableT* src = table + (size_t)id * width;
-    for (int c = threadIdx.x; c < width; c += blockDim.x) dst[c] = to_f32(src[c]) * scale;
 }
 
 template <typename TableT>
@@ -106,13 +106,13 @@ __global__ void stream_entry_kernel(float* __restrict__ x, const float* __restri
 }  // namespace
 
 MLB_EXPORT int mlb_embed_gather_scaled(const void* table, int table_dtype, const int* ids, float* out, int tokens, int width,
-                                       int vocab, float scale, cudaStream_t stream) {
-    if (tokens < 0 || width <= 0 || vocab <= 0) return fail(MLB_INVALID_ARGUMENT, "embed_gather_scaled: bad sizes");
+                                       int vocab, float scale, int copies, cudaStream_t stream) {
+    if (tokens < 0 || width <= 0 || vocab <= 0 || copies <= 0) return fail(MLB_INVALID_ARGUMENT, "embed_gather_scaled: bad sizes");
     if (tokens == 0) return MLB_OK;
     if (table_dtype == MLB_F32)
-        launch_kernel(embed_scaled_kernel<float>, tokens, ROW_THREADS, 0, stream, (const float*)table, ids, out, tokens, width, vocab, scale);
+        launch_kernel(embed_scaled_kernel<float>, tokens, ROW_THREADS, 0, stream, (const float*)table, ids, out, tokens, width, vocab, scale, copies);
     else if (table_dtype == MLB_BF16)
-        launch_kernel(embed_scaled_kernel<__nv_bfloat16>, tokens, ROW_THREADS, 0, stream, (const __nv_bfloat16*)table, ids, out, tokens, width, vocab, scale);
+        launch_kernel(embed_scaled_kernel<__nv_bfloat16>, tokens, ROW_THREADS, 0, stream, (const __nv_bfloat16*)table, ids, out, tokens, width, vocab, scale, copies);
     else
         return fail(MLB_INVALID_ARGUMENT, "embed_gather_scaled: unknown table dtype %d", table_dtype);
     return check_launch("embed_gather_scaled");

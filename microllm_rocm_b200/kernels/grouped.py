@@ -26,7 +26,7 @@ MMA_SOURCE = "grouped_mma.cu"
 ops.register_signatures(MMA_SOURCE, {
     "mlb_grouped_mma": [c_void_p, c_longlong, c_longlong, c_void_p, c_longlong, c_longlong, c_void_p, c_longlong, c_longlong,
                         c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_longlong, c_int, c_int, c_int, c_int, c_int,
-                        c_int, c_void_p],
+                        c_int, c_int, c_void_p],
 })
 
 # Tests set it to False to send bf16 products to the CUDA-core kernel and compare.
@@ -88,7 +88,7 @@ def grouped_linear(a: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, *, 
             a.data_ptr(), a.stride(0), a_group_cols, weight.data_ptr(), weight.stride(1), weight.stride(0), out.data_ptr(),
             out.stride(0), c_group_cols, ops._ptr(group_offsets), ops._ptr(a_rows), ops._ptr(c_rows), int(a_row_div),
             ops._ptr(factor), factor.stride(0) if factor is not None else 0, 0, int(rows), N, K, G, ops.dtype_tag(out),
-            int(row_tile), ops._stream()))
+            int(row_tile), 0, ops._stream()))
         return
     L = ops.lib(SOURCE)
     build.check(L, L.mlb_grouped_gemm(
@@ -99,13 +99,17 @@ def grouped_linear(a: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, *, 
 
 
 def grouped_silu_mul(a: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, *, rows: int, group_offsets: torch.Tensor,
-                     a_rows: Optional[torch.Tensor] = None, a_row_div: int = 1, row_tile: int = 64, alloc=None) -> None:
-    """weight [G, 2 * F, K]: per group F gate rows over F up rows; out[place] = silu(a gate^T) * (a up^T), [rows, F].
+                     a_rows: Optional[torch.Tensor] = None, a_row_div: int = 1, row_tile: int = 64, alloc=None,
+                     activation: str = "silu", limit: Optional[float] = None) -> None:
+    """weight [G, 2 * F, K]: per group F gate rows over F up rows; out[place] = silu(a gate^T) * (a up^T), [rows, F]; or,
+    with `activation` "clamped_swish" and its `limit`, the clamped form (ops.activation_code).
     On the tensor cores both products and the activation are one kernel; otherwise the fused product leaves
     [rows, 2 * F] (from `alloc(shape, dtype)`) and the activation kernel follows."""
     ops._need(a, "a", dims=2); ops._need(weight, "weight", dims=3); ops._need(out, "out", dims=2)
     G, two_f, K = weight.shape
     F = two_f // 2
+    if activation not in ("silu", ops.CLAMPED_ACTIVATION):
+        raise KernelError(f"grouped_silu_mul: activation {activation!r}")
     if two_f % 2 or tuple(out.shape) != (rows, F):
         raise KernelError("grouped_silu_mul: the weight holds gate rows over up rows, the output one column per pair")
     if mma_supported(a, weight):
@@ -116,9 +120,9 @@ def grouped_silu_mul(a: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, *
         build.check(L, L.mlb_grouped_mma(
             a.data_ptr(), a.stride(0), 0, weight.data_ptr(), weight.stride(1), weight.stride(0), out.data_ptr(), out.stride(0), 0,
             group_offsets.data_ptr(), ops._ptr(a_rows), None, int(a_row_div), None, 0, F, int(rows), F, K, G,
-            ops.dtype_tag(out), int(row_tile), ops._stream()))
+            ops.dtype_tag(out), int(row_tile), ops.activation_code(activation, limit), ops._stream()))
         return
     row_tile = min(row_tile, 64)
     gate_up = alloc((rows, two_f), a.dtype) if alloc is not None else torch.empty((rows, two_f), dtype=a.dtype, device=a.device)
     grouped_linear(a, weight, gate_up, rows=rows, group_offsets=group_offsets, a_rows=a_rows, a_row_div=a_row_div, row_tile=row_tile)
-    ops.silu_mul(gate_up, out)
+    ops.gated_act_mul(gate_up, out, activation, limit)

@@ -24,8 +24,11 @@ ops.register_signatures("linear_attention.cu", {
                           c_void_p, c_longlong, c_int, c_longlong, c_int, c_float, c_void_p, c_longlong, c_int, c_longlong, c_int,
                           c_int, c_int, c_void_p, c_void_p, c_longlong, c_int, c_longlong, c_void_p, c_int, c_float, c_void_p,
                           c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
-    "mlb_head_norm_gate": [c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_int, c_longlong, c_int, c_int, c_void_p, c_int, c_int,
-                           c_int, c_int, c_float, c_void_p],
+    "mlb_head_norm_gate": [c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_int, c_longlong, c_int, c_int, c_void_p, c_void_p, c_float,
+                           c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p],
+    "mlb_head_decay_prepare": [c_void_p, c_longlong, c_int, c_longlong, c_int, c_int, c_int, c_void_p, c_int, c_float, c_float, c_void_p, c_void_p,
+                               c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_int,
+                               c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p],
     "mlb_lightning_prepare": [c_void_p, c_longlong, c_int, c_longlong, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                               c_int, c_int, c_int, c_int, c_void_p],
     "mlb_row_norm_gate": [c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_longlong, c_int, c_void_p, c_int, c_int, c_int, c_float, c_void_p],
@@ -92,9 +95,10 @@ def decay_prepare(q_src, q_col: int, k_src, k_col: int, v_src, v_col: int, q_sca
 
 
 def head_norm_gate(o: torch.Tensor, weight: Optional[torch.Tensor], gate, gate_col: int, gate_act: str, out: torch.Tensor, heads: int,
-                   dv: int, eps: float) -> None:
+                   dv: int, eps: float, den: Optional[torch.Tensor] = None, floor: Optional[torch.Tensor] = None, den_eps: float = 0.0) -> None:
     """out = o / rms(o) per head * weight * act(gate columns from gate_col) in out's dtype; `weight` [dv] (shared by the
-    heads), [heads * dv] or None; `gate` fp32 rows or partial results, or None."""
+    heads), [heads * dv] or None; `gate` fp32 rows or partial results, or None.  With `den` and `floor` [T, heads] fp32 a
+    head's o is first divided by max(|den|, floor) + den_eps."""
     ops._need(o, "o", torch.float32, 2); ops._need(out, "out", dims=2)
     T = o.shape[0]
     if o.shape != (T, heads * dv) or out.shape != o.shape or not 0 < dv <= MAX_WIDTH:
@@ -107,13 +111,21 @@ def head_norm_gate(o: torch.Tensor, weight: Optional[torch.Tensor], gate, gate_c
         if weight.shape[0] not in (dv, heads * dv):
             raise KernelError("head_norm_gate: the weight must have dv or heads * dv elements")
         per_head = 1 if weight.shape[0] == heads * dv and heads > 1 else 0
+    for name, t in (("den", den), ("floor", floor)):
+        if t is not None:
+            ops._need(t, name, torch.float32, 2)
+            if tuple(t.shape) != (T, heads):
+                raise KernelError(f"head_norm_gate: {name} must be [T, heads]")
+    if (den is None) != (floor is None):
+        raise KernelError("head_norm_gate: den and floor come together")
     g_ptr, g_ld, g_n, g_stride = None, 0, 1, 0
     if gate is not None:
         _, g_ld, g_n, g_stride = _columns(gate, "gate")
         g_ptr = gate.data_ptr()
     L = ops.lib("linear_attention.cu")
     build.check(L, L.mlb_head_norm_gate(o.data_ptr(), ops._ptr(weight), per_head, g_ptr, g_ld, g_n, g_stride, int(gate_col),
-                                        GATE_ACTS[gate_act], out.data_ptr(), ops.dtype_tag(out), T, heads, dv, float(eps), ops._stream()))
+                                        GATE_ACTS[gate_act], ops._ptr(den), ops._ptr(floor), float(den_eps), out.data_ptr(), ops.dtype_tag(out), T,
+                                        heads, dv, float(eps), ops._stream()))
 
 
 def lightning_prepare(proj, q_col: int, k_col: int, v_col: int, head_decay: torch.Tensor, q_out: torch.Tensor, k_out: torch.Tensor,
@@ -155,3 +167,43 @@ def row_norm_gate(o: torch.Tensor, weight: Optional[torch.Tensor], gate, gate_co
     L = ops.lib("linear_attention.cu")
     build.check(L, L.mlb_row_norm_gate(o.data_ptr(), ops._ptr(weight), g_ptr, g_ld, g_n, g_stride, int(gate_col), out.data_ptr(),
                                        ops.dtype_tag(out), T, width, float(eps), ops._stream()))
+
+
+def head_decay_prepare(proj, q_col: int, k_col: int, v_col: int, q_out: torch.Tensor, k_out: torch.Tensor, v_out: torch.Tensor, heads: int,
+                       dk: int, dv: int, ctx, q_scale: float = 1.0, k_scale: float = 1.0, cos_sin: Optional[torch.Tensor] = None,
+                       gates: Optional[torch.Tensor] = None, i_col: int = 0, f_col: int = 0, i_bias: Optional[torch.Tensor] = None,
+                       f_bias: Optional[torch.Tensor] = None, cap: float = 1.0, m_state: Optional[torch.Tensor] = None,
+                       slots: Optional[torch.Tensor] = None) -> None:
+    """q_out = q * q_scale, k_out = k * k_scale [T, heads * dk], v_out [T, heads * dv] out of the column blocks of `proj` (fp32 rows
+    or partial results); with `cos_sin` [T, pairs, 2] the first 2 * pairs elements of every head of q and k are turned in front
+    of the scale (element i with i + pairs).  With `gates` [3, T, heads] fp32 also the gates of a matrix memory with exponential
+    gates, from columns i_col + h and f_col + h and the biases [heads]: i = cap tanh((a + b) / cap), f the log sigmoid of the
+    same form, m_t = max(f + m_(t-1), i) carried in `m_state` [slots, heads] (0 at position 0);
+    gates = exp(f + m_(t-1) - m_t), exp(i - m_t), exp(-m_t)."""
+    _, ld, n, stride = _columns(proj, "proj")
+    T = proj.shape[-2]
+    for name, t, shape in (("q_out", q_out, (T, heads * dk)), ("k_out", k_out, (T, heads * dk)), ("v_out", v_out, (T, heads * dv))):
+        ops._need(t, name, torch.float32, 2)
+        if tuple(t.shape) != shape:
+            raise KernelError(f"head_decay_prepare: {name} must be {shape}")
+    if max(q_col, k_col) + heads * dk > ld or v_col + heads * dv > ld:
+        raise KernelError("head_decay_prepare: shapes do not agree")
+    rot = 0
+    if cos_sin is not None:
+        ops._need(cos_sin, "cos_sin", torch.float32, 3)
+        rot = 2 * cos_sin.shape[1]
+        if tuple(cos_sin.shape) != (T, rot // 2, 2) or rot > dk:
+            raise KernelError("head_decay_prepare: cos_sin must be [T, pairs, 2] with at most dk / 2 pairs")
+    gate_args = [0, 0, None, None, 1.0, None, None, 0, None, None, 0, None]
+    if gates is not None:
+        ops._need(gates, "gates", torch.float32, 3); ops._need(m_state, "m_state", torch.float32, 2)
+        ops._need(i_bias, "i_bias", torch.float32, 1); ops._need(f_bias, "f_bias", torch.float32, 1)
+        if tuple(gates.shape) != (3, T, heads) or m_state.shape[1] != heads or i_bias.shape[0] != heads or f_bias.shape[0] != heads \
+                or max(i_col, f_col) + heads > ld:
+            raise KernelError("head_decay_prepare: the gates' shapes do not agree")
+        gate_args = [int(i_col), int(f_col), i_bias.data_ptr(), f_bias.data_ptr(), float(cap), m_state.data_ptr(), slots.data_ptr(),
+                     m_state.shape[0], ctx.seq_starts.data_ptr(), ctx.seq_pos0.data_ptr(), ctx.num_seqs, gates.data_ptr()]
+    L = ops.lib("linear_attention.cu")
+    build.check(L, L.mlb_head_decay_prepare(proj.data_ptr(), ld, n, stride, int(q_col), int(k_col), int(v_col), ops._ptr(cos_sin), rot,
+                                            float(q_scale), float(k_scale), q_out.data_ptr(), k_out.data_ptr(), v_out.data_ptr(), T, heads,
+                                            dk, dv, *gate_args, ops._ptr(ctx.error_flag), ops._stream()))

@@ -2,7 +2,7 @@
 (token, choice) pairs sorted by expert; the weighted sum of the experts' results."""
 from __future__ import annotations
 
-from ctypes import c_int, c_longlong, c_void_p
+from ctypes import c_float, c_int, c_longlong, c_void_p
 from typing import Optional
 
 import torch
@@ -13,14 +13,14 @@ from .build import KernelError
 SOURCE = "moe.cu"
 ops.register_signatures(SOURCE, {
     "mlb_moe_select": [c_void_p, c_longlong, c_int, c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p,
-                       c_int, c_void_p],
+                       c_int, c_int, c_int, c_float, c_void_p],
     "mlb_moe_align": [c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p],
     "mlb_moe_combine": [c_void_p, c_void_p, c_void_p, c_int, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
                         c_void_p, c_int, c_void_p, c_int, c_void_p],
 })
 
 
-SCORINGS = {"top_softmax": 0, "softmax_all": 1}
+SCORINGS = {"top_softmax": 0, "softmax_all": 1, "sigmoid_groups": 2}
 
 
 def sources():
@@ -28,12 +28,16 @@ def sources():
 
 
 def select(logits: torch.Tensor, experts: int, bias: Optional[torch.Tensor], top: int, ids: torch.Tensor, weights: torch.Tensor,
-           gate_col: int = -1, gate_out: Optional[torch.Tensor] = None, scoring: str = "top_softmax") -> None:
+           gate_col: int = -1, gate_out: Optional[torch.Tensor] = None, scoring: str = "top_softmax",
+           groups: int = 1, keep: int = 1, weight_scale: float = 1.0) -> None:
     """logits [T, N] fp32 (or [S, T, N] partial sums of a split product), N >= experts: the router's logits in the first
     `experts` columns, bias [experts] fp32 added here.  ids [T, top] int32 and weights [T, top] fp32 receive the chosen
     experts in order of their logits and the softmax over the chosen logits.  gate_col >= 0 and gate_out [T] fp32:
     sigmoid of that column per token.  `scoring` "softmax_all": s = softmax over all `experts` columns, the choice goes by
-    s + bias (a correction that only steers the choice) and the weights are the chosen s, not renormalised."""
+    s + bias (a correction that only steers the choice) and the weights are the chosen s, not renormalised.  "sigmoid_groups":
+    s = sigmoid of every column; the experts form `groups` equal groups of neighbours, a group scores the sum of its two largest
+    s + bias, only experts of the `keep` best groups can be chosen (ties: the smaller index), and the weights are the chosen s
+    divided by their sum + 1e-20, times `weight_scale`."""
     if scoring not in SCORINGS:
         raise KernelError(f"moe.select: scoring {scoring!r} is not one of {', '.join(SCORINGS)}")
     n_partials, stride, first = 1, 0, logits
@@ -58,7 +62,7 @@ def select(logits: torch.Tensor, experts: int, bias: Optional[torch.Tensor], top
     L = ops.lib(SOURCE)
     build.check(L, L.mlb_moe_select(first.data_ptr(), first.stride(0), n_partials, stride, ops._ptr(bias), int(gate_col), T,
                                     int(experts), int(top), ids.data_ptr(), weights.data_ptr(), ops._ptr(gate_out), SCORINGS[scoring],
-                                    ops._stream()))
+                                    int(groups), int(keep), float(weight_scale), ops._stream()))
 
 
 def align(ids: torch.Tensor, experts: int, offsets: torch.Tensor, sorted_pairs: torch.Tensor,

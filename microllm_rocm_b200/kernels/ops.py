@@ -85,7 +85,7 @@ _SIGNATURES = {
                                       c_float, c_void_p, c_void_p],
     },
     "residual.cu": {
-        "mlb_embed_gather_scaled": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_void_p],
+        "mlb_embed_gather_scaled": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_int, c_void_p],
         "mlb_add_table_rows": [c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p],
         "mlb_add_scaled_rmsnorm": [c_void_p, c_void_p, c_int, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
                                    c_float, c_void_p],
@@ -99,6 +99,11 @@ _SIGNATURES = {
         "mlb_layernorm": [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_float, c_void_p],
         "mlb_scale_add_layernorm": [c_void_p, c_float, c_void_p, c_int, c_longlong, c_float, c_void_p, c_int, c_longlong, c_float,
                                     c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_void_p],
+    },
+    "streams.cu": {
+        "mlb_streams_mix_norm": [c_void_p, c_void_p, c_int, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int,
+                                 c_void_p, c_int, c_int, c_int, c_float, c_void_p],
+        "mlb_streams_total": [c_void_p, c_void_p, c_int, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
     },
     "post_norm.cu": {
         "mlb_normed_add_rmsnorm": [c_void_p, c_void_p, c_int, c_longlong, c_float, c_void_p, c_int, c_longlong, c_float, c_void_p,
@@ -166,7 +171,7 @@ def part_sources():
     `kernel_sources`)."""
     return [("residual.cu", {}), ("grouped_gemm.cu", {}), ("grouped_mma.cu", {}), ("latent.cu", {}), ("moe.cu", {}),
             ("layernorm.cu", {}), ("short_conv.cu", {}), ("attention_kv.cu", {}), ("delta_rule.cu", {}),
-            ("linear_attention.cu", {}), ("post_norm.cu", {})]
+            ("linear_attention.cu", {}), ("post_norm.cu", {}), ("streams.cu", {})]
 
 
 def all_sources():
@@ -365,31 +370,38 @@ def copy_raw(dst: int, src: int, nbytes: int, to_device: bool) -> None:
 
 
 # ------------------------------------------------------------------------------ layer norm
-def layernorm(x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor, eps: float, out: torch.Tensor,
+def _need_bias(bias: Optional[torch.Tensor], width: int, what: str) -> None:
+    if bias is not None:
+        _need(bias, "bias", torch.float32, 1)
+        if bias.shape[0] != width:
+            raise KernelError(f"{what}: shapes do not agree")
+
+
+def layernorm(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor], eps: float, out: torch.Tensor,
               rows: Optional[torch.Tensor] = None) -> None:
-    """out[r] = (v - mean) / sqrt(var + eps) * weight + bias with v = x[rows[r]] if rows is given else x[r]; fp32 math."""
-    _need(x, "x", torch.float32, 2); _need(weight, "weight", torch.float32, 1); _need(bias, "bias", torch.float32, 1)
+    """out[r] = (v - mean) / sqrt(var + eps) * weight (+ bias) with v = x[rows[r]] if rows is given else x[r]; fp32 math."""
+    _need(x, "x", torch.float32, 2); _need(weight, "weight", torch.float32, 1); _need_bias(bias, x.shape[1], "layernorm")
     _need(out, "out", dims=2)
     width = x.shape[1]
     n = rows.shape[0] if rows is not None else x.shape[0]
     if rows is not None:
         _need(rows, "rows", torch.int32, 1)
-    if weight.shape[0] != width or bias.shape[0] != width or out.shape != (n, width):
+    if weight.shape[0] != width or out.shape != (n, width):
         raise KernelError("layernorm: shapes do not agree")
     L = lib("layernorm.cu")
-    build.check(L, L.mlb_layernorm(x.data_ptr(), weight.data_ptr(), bias.data_ptr(), out.data_ptr(), dtype_tag(out), _ptr(rows),
+    build.check(L, L.mlb_layernorm(x.data_ptr(), weight.data_ptr(), _ptr(bias), out.data_ptr(), dtype_tag(out), _ptr(rows),
                                    n, width, float(eps), _stream()))
 
 
-def scale_add_layernorm(x: torch.Tensor, alpha: float, terms, weight: torch.Tensor, bias: torch.Tensor, eps: float,
+def scale_add_layernorm(x: torch.Tensor, alpha: float, terms, weight: torch.Tensor, bias: Optional[torch.Tensor], eps: float,
                         out: Optional[torch.Tensor]) -> None:
     """x <- layernorm(alpha * x + sum_i s_i * d_i) in place (fp32), and `out` (when given) a copy of the new x in its own
     dtype.  `terms`: one or two (s_i, d_i); a d_i may be [S, M, N] partial results, summed over S in order."""
-    _need(x, "x", torch.float32, 2); _need(weight, "weight", torch.float32, 1); _need(bias, "bias", torch.float32, 1)
+    _need(x, "x", torch.float32, 2); _need(weight, "weight", torch.float32, 1); _need_bias(bias, x.shape[1], "scale_add_layernorm")
     terms = list(terms)
     if not 1 <= len(terms) <= 2:
         raise KernelError("scale_add_layernorm: one or two terms")
-    if weight.shape[0] != x.shape[1] or bias.shape[0] != x.shape[1]:
+    if weight.shape[0] != x.shape[1]:
         raise KernelError("scale_add_layernorm: shapes do not agree")
     if out is not None:
         _need(out, "out", dims=2)
@@ -402,7 +414,7 @@ def scale_add_layernorm(x: torch.Tensor, alpha: float, terms, weight: torch.Tens
     if len(terms) == 1:
         args += [None, 0, 0, 0.0]
     L = lib("layernorm.cu")
-    build.check(L, L.mlb_scale_add_layernorm(x.data_ptr(), float(alpha), *args, weight.data_ptr(), bias.data_ptr(), _ptr(out),
+    build.check(L, L.mlb_scale_add_layernorm(x.data_ptr(), float(alpha), *args, weight.data_ptr(), _ptr(bias), _ptr(out),
                                              dtype_tag(out) if out is not None else F32, x.shape[0], x.shape[1], float(eps),
                                              _stream()))
 
@@ -433,16 +445,66 @@ def normed_add_rmsnorm(x: torch.Tensor, terms, post_weight: torch.Tensor, eps: f
                                             _stream()))
 
 
+# ------------------------------------------------------------------------------ several residual streams
+MAX_STREAMS = 16
+
+
+def _stream_args(x: torch.Tensor, pending, what: str):
+    """(rows, streams, width) and the launcher's arguments for a pending result: None or (y, mix [S, S], out [S]), y [T, W]
+    fp32 or its [K, T, W] partial results."""
+    _need(x, "x", torch.float32, 3)
+    T, S, W = x.shape
+    if not 0 < S <= MAX_STREAMS:
+        raise KernelError(f"{what}: {S} streams (at most {MAX_STREAMS})")
+    if pending is None:
+        return T, S, W, [None, 0, 0, None, None]
+    y, mix, out_w = pending
+    n, stride = _partials(y, (T, W), f"{what} pending result")
+    _need(mix, "mix", torch.float32, 2); _need(out_w, "out_w", torch.float32, 1)
+    if tuple(mix.shape) != (S, S) or out_w.shape[0] != S:
+        raise KernelError(f"{what}: shapes do not agree")
+    return T, S, W, [y.data_ptr(), n, stride, mix.data_ptr(), out_w.data_ptr()]
+
+
+def streams_mix_norm(x: torch.Tensor, pending, in_w: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor], eps: float,
+                     centred: bool, out: torch.Tensor, rows: Optional[torch.Tensor] = None) -> None:
+    """x [T, S, W] fp32: with a pending (y, mix, out_w), x[:, t] <- sum_s mix[s, t] x[:, s] + out_w[t] * y in place; then
+    out = norm(sum_s in_w[s] * x[:, s]) * weight (+ bias), a layer norm (`centred`) or an rms norm.  With `rows` only those
+    rows are made and the streams stay as they are."""
+    T, S, W, args = _stream_args(x, pending, "streams_mix_norm")
+    _need(in_w, "in_w", torch.float32, 1); _need(weight, "weight", torch.float32, 1); _need_bias(bias, W, "streams_mix_norm")
+    _need(out, "out", dims=2)
+    if rows is not None:
+        _need(rows, "rows", torch.int32, 1)
+    n = rows.shape[0] if rows is not None else T
+    if in_w.shape[0] != S or weight.shape[0] != W or tuple(out.shape) != (n, W):
+        raise KernelError("streams_mix_norm: shapes do not agree")
+    L = lib("streams.cu")
+    build.check(L, L.mlb_streams_mix_norm(x.data_ptr(), *args, in_w.data_ptr(), weight.data_ptr(), _ptr(bias), 1 if centred else 0,
+                                          out.data_ptr(), dtype_tag(out), _ptr(rows), n, S, W, float(eps), _stream()))
+
+
+def streams_total(x: torch.Tensor, pending, out: torch.Tensor) -> None:
+    """out [T, W] fp32 = the sum of the streams with a pending result taken in; x stays as it is."""
+    T, S, W, args = _stream_args(x, pending, "streams_total")
+    _need(out, "out", torch.float32, 2)
+    if tuple(out.shape) != (T, W):
+        raise KernelError("streams_total: shapes do not agree")
+    L = lib("streams.cu")
+    build.check(L, L.mlb_streams_total(x.data_ptr(), *args, out.data_ptr(), T, S, W, _stream()))
+
+
 # ------------------------------------------------------------------------------ scaled residual stream
 def embed_gather_scaled(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor, scale: float) -> None:
-    """out[t] = table[ids[t]] * scale (fp32)."""
-    _need(table, "table", dims=2); _need(ids, "ids", torch.int32, 1); _need(out, "out", torch.float32, 2)
+    """out[t] = table[ids[t]] * scale (fp32); `out` [T, width], or [T, copies, width]: every copy the same row."""
+    _need(table, "table", dims=2); _need(ids, "ids", torch.int32, 1); _need(out, "out", torch.float32)
     vocab, width = table.shape
-    if out.shape != (ids.shape[0], width):
+    copies = out.shape[1] if out.dim() == 3 else 1
+    if out.shape not in ((ids.shape[0], width), (ids.shape[0], copies, width)):
         raise KernelError(f"embed_gather_scaled: out {tuple(out.shape)} does not match ({ids.shape[0]}, {width})")
     L = lib("residual.cu")
     build.check(L, L.mlb_embed_gather_scaled(table.data_ptr(), dtype_tag(table), ids.data_ptr(), out.data_ptr(),
-                                             ids.shape[0], width, vocab, float(scale), _stream()))
+                                             ids.shape[0], width, vocab, float(scale), copies, _stream()))
 
 
 def add_table_rows(x: torch.Tensor, table: torch.Tensor, index: torch.Tensor) -> None:
@@ -691,6 +753,31 @@ def rope_table(positions: torch.Tensor, inv_freq: torch.Tensor, out: Optional[to
 
 
 # ------------------------------------------------------------------------------ attention
+DISTANCE_PAD = 256          # csrc/common.cuh: DISTANCE_PAD
+
+
+class DistanceBias:
+    """What is added to a score by head and distance query - key, as the attention kernels read it: `values` [heads, n] holds
+    distances 0..n-1, every larger distance takes the last one's.  The table on the device repeats the first value in front
+    and the last one behind, so that a tile of distances may run over either end."""
+
+    def __init__(self, values: torch.Tensor):
+        values = values.to(torch.float32)
+        self.heads, n = values.shape
+        self.last = n - 1
+        pad = lambda column: values[:, column:column + 1].expand(-1, DISTANCE_PAD)
+        self.table = torch.cat([pad(0), values, pad(n - 1)], 1).contiguous()
+
+
+def distance_bias_args(bias: Optional[DistanceBias], heads: int):
+    if bias is None:
+        return (None, 0)
+    _need(bias.table, "distance bias", torch.float32, 2)
+    if bias.heads != heads:
+        raise KernelError(f"the distance bias has {bias.heads} heads, the attention {heads}")
+    return (bias.table.data_ptr(), bias.last)
+
+
 def paged_attention_plain(q: torch.Tensor, pages: torch.Tensor, out: torch.Tensor, positions: torch.Tensor,
                           token_seq: torch.Tensor, block_table: torch.Tensor, num_heads: int, num_kv_heads: int,
                           head_dim: int, scale: float, window: Optional[int],

@@ -28,6 +28,8 @@ ops.register_signatures("delta_rule.cu", {
     "mlb_take_columns": [c_void_p, c_longlong, c_int, c_longlong, c_int, c_int, c_int, c_void_p, c_int, c_int, c_void_p],
     "mlb_linear_scan": [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int,
                         c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
+    "mlb_head_scan": [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
+                      c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
     "mlb_delta_scan": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
                        c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
     "mlb_delta_output": [c_void_p, c_void_p, c_void_p, c_longlong, c_int, c_longlong, c_int, c_void_p, c_void_p, c_longlong, c_int,
@@ -180,3 +182,38 @@ def linear_scan(rule: str, q: torch.Tensor, k: torch.Tensor, decay: torch.Tensor
     build.check(L, L.mlb_linear_scan(RULES[rule], q.data_ptr(), k.data_ptr(), decay.data_ptr(), ops._ptr(bonus), v.data_ptr(), v.stride(0),
                                      o.data_ptr(), state.data_ptr(), slots.data_ptr(), state.shape[0], ctx.seq_starts.data_ptr(),
                                      ctx.seq_pos0.data_ptr(), ctx.num_seqs, heads, heads, dk, dv, ops._ptr(ctx.error_flag), ops._stream()))
+
+
+def head_scan(q: torch.Tensor, k: torch.Tensor, decay: torch.Tensor, v: torch.Tensor, o: torch.Tensor, state: torch.Tensor,
+              slots: torch.Tensor, ctx, heads: int, dk: int, dv: int, weight: Optional[torch.Tensor] = None,
+              n_state: Optional[torch.Tensor] = None, den: Optional[torch.Tensor] = None) -> None:
+    """A recurrence with one decay per head over the step's tokens, per head with S [dk, dv]:
+      S <- decay_t S + weight_t k_t v_t^T;  o_t = S^T q_t
+    `decay` [T, heads], or [heads]: one fixed number per head; `weight` [T, heads] or None (1).  With `n_state`
+    [slots, heads, dk] and `den` [T, heads] a vector runs beside S: n <- decay_t n + weight_t k_t, den_t = n . q_t.
+    q, k [T, heads * dk], v, o [T, heads * dv] fp32; states fp32, taken as zero for a sequence that starts at position 0."""
+    T = q.shape[0]
+    for name, t, shape in (("q", q, (T, heads * dk)), ("k", k, (T, heads * dk)), ("v", v, (T, heads * dv)), ("o", o, (T, heads * dv))):
+        ops._need(t, name, torch.float32, 2)
+        if tuple(t.shape) != shape:
+            raise KernelError(f"head_scan: {name} must be {shape}, got {tuple(t.shape)}")
+    per_token = decay.dim() == 2
+    for name, t, shape in (("decay", decay, (T, heads) if per_token else (heads,)), ("weight", weight, (T, heads)), ("den", den, (T, heads))):
+        if t is not None:
+            ops._need(t, name, torch.float32)
+            if tuple(t.shape) != shape:
+                raise KernelError(f"head_scan: {name} must be {shape}, got {tuple(t.shape)}")
+    if (n_state is None) != (den is None):
+        raise KernelError("head_scan: the vector's state and its read-out come together")
+    ops._need(state, "state", torch.float32, 4)
+    if tuple(state.shape[1:]) != (heads, dk, dv):
+        raise KernelError(f"head_scan: the state must be [slots, {heads}, {dk}, {dv}], got {tuple(state.shape)}")
+    if n_state is not None:
+        ops._need(n_state, "n_state", torch.float32, 3)
+        if tuple(n_state.shape) != (state.shape[0], heads, dk):
+            raise KernelError(f"head_scan: the vector's state must be [{state.shape[0]}, {heads}, {dk}], got {tuple(n_state.shape)}")
+    L = ops.lib("delta_rule.cu")
+    build.check(L, L.mlb_head_scan(q.data_ptr(), k.data_ptr(), decay.data_ptr(), 1 if per_token else 0, ops._ptr(weight), v.data_ptr(), v.stride(0),
+                                   o.data_ptr(), state.data_ptr(), ops._ptr(n_state), ops._ptr(den), slots.data_ptr(), state.shape[0],
+                                   ctx.seq_starts.data_ptr(), ctx.seq_pos0.data_ptr(), ctx.num_seqs, heads, dk, dv, ops._ptr(ctx.error_flag),
+                                   ops._stream()))

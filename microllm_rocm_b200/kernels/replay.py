@@ -24,7 +24,7 @@ def _register():
                              c_float, c_int, c_void_p],
     })
 
-MAX_SLOTS = 28
+MAX_SLOTS = 32
 MAX_FLOATS = 4
 
 

@@ -27,6 +27,18 @@ ROPE_TABLE_MIN_TOKENS = 64          # from here on a step-wide table of sines an
 SHARED_KERNEL_WIDTHS = (32, 64, 128, 256)   # head sizes at which the tensor-core attention kernels of one width are built and tested
 
 
+def distance_rows(buckets: int, far: float):
+    """The row of a table of `buckets` rows that each distance 0, 1, .. reads, up to the first distance that reads the last row
+    (as all larger ones do): distances below buckets // 2 have a row each, from there on
+    near + floor(ln(n / near) / ln(far / near) * (buckets - near)), near = buckets // 2, at most buckets - 1."""
+    near = buckets // 2
+    rows = list(range(near))
+    while not rows or rows[-1] != buckets - 1:
+        n = len(rows)
+        rows.append(min(buckets - 1, near + int(math.floor(math.log(n / near) / math.log(far / near) * (buckets - near)))))
+    return rows
+
+
 @register_mixer("attention")
 class Attention(Mixer):
     graph_safe = True
@@ -172,6 +184,8 @@ class NormedAttention(Mixer):
     Further options: `bias` (q and k projections have biases, added as the projection is read; values that are the projected
     keys carry the key's bias), `qk_norm="row"` (q and k are each divided by the root mean square of their WHOLE projection
     row, before the split into heads, times a weight of the row's length), `softcap` (score <- cap * tanh(score / cap)),
+    `distance_bias` {buckets, far} (score + R[bucket(query - key), head] with a learned table R of `buckets` rows: distances below
+    buckets // 2 have a row each, from there on the rows widen logarithmically up to `far`; neither scaled nor capped),
     `sink` ("learned": one number per head whose exponential joins the softmax's denominator, with no key and no value,
     neither scaled nor capped; "zero": the same with the number fixed at 0, i.e. 1 is added to the denominator), and
     `kv_shared` (the layer has no key and value projections of its own: its run reads the pages another run wrote, with its
@@ -202,6 +216,10 @@ class NormedAttention(Mixer):
         if self.sink_kind not in (None, "learned", "zero"):
             raise ValueError(f"normed_attention: sink {self.sink_kind!r} is not 'learned' or 'zero'")
         self.kv_shared = bool(params.get("kv_shared", False))
+        bias = params.get("distance_bias")
+        self.distance = (int(bias["buckets"]), float(bias["far"])) if bias else None
+        if self.distance and not self.distance[1] > self.distance[0] // 2 > 0:
+            raise ValueError("normed_attention: a distance bias needs two rows or more and `far` beyond half of them")
         self.q_temp = tuple(params["q_temp"]) if params.get("q_temp") else None
         self.window = params.get("window")
         self.chunk = int(params["chunk"]) if params.get("chunk") else None
@@ -224,7 +242,7 @@ class NormedAttention(Mixer):
             raise ValueError("normed_attention: biases and a convolution do not go together")
         names = dict(q="q_proj.weight", k="k_proj.weight", v="v_proj.weight", o="o_proj.weight", q_norm="q_norm.weight",
                      k_norm="k_norm.weight", gate="g_proj.weight", q_conv="q_conv.weight", k_conv="k_conv.weight",
-                     v_conv="v_conv.weight", q_bias="q_proj.bias", k_bias="k_proj.bias", sink="sink")
+                     v_conv="v_conv.weight", q_bias="q_proj.bias", k_bias="k_proj.bias", sink="sink", distance="distance_bias.weight")
         names.update(params.get("names", {}))
         self.names = names
         self.rt = rt
@@ -247,7 +265,7 @@ class NormedAttention(Mixer):
             self.stored = next((w for w in SHARED_KERNEL_WIDTHS if w >= max(self.dk, self.dv)), None)
         if self.stored is not None and not attention_kernels.extras_supported(self.stored, self.softcap, self.sink_kind is not None):
             self.stored = None           # a cap or a sink that the kernels of one width do not take: the plain kernel
-        self.w_in = self.w_o = self.q_norm_w = self.k_norm_w = self.w_conv = self.b_in = self.sink = None
+        self.w_in = self.w_o = self.q_norm_w = self.k_norm_w = self.w_conv = self.b_in = self.sink = self.bias = None
         # rows of the fused projection; a gate of one row per head is padded to a multiple of 8 rows, which the products like
         self.in_rows = -(-(self.conv_cols + self.g_cols) // 8) * 8 if self.gate_per_head else self.conv_cols + self.g_cols
 
@@ -283,6 +301,8 @@ class NormedAttention(Mixer):
                 specs[n["k_norm"]] = WeightSpec((self.k_cols,), role="vector", init=("one_plus_normal", 0.1))
         if self.sink_kind == "learned":
             specs[n["sink"]] = WeightSpec((self.nh,), role="vector", init=("normal", 1.0))
+        if self.distance:
+            specs[n["distance"]] = WeightSpec((self.distance[0], self.nh), role="vector", init=("normal", 0.5))
         if self.v_cols:
             specs[n["v"]] = WeightSpec((self.v_cols, self.hidden))
         if self.has_gate:
@@ -342,6 +362,9 @@ class NormedAttention(Mixer):
             self.sink = tensors[n["sink"]]
         elif self.sink_kind == "zero":
             self.sink = torch.zeros((self.nh,), dtype=torch.float32, device=self.w_in.device)
+        if self.distance:                                # the rows spread over the distances once: [heads, distances]
+            rows = torch.tensor(distance_rows(*self.distance), dtype=torch.long, device=self.w_in.device)
+            self.bias = ops.DistanceBias(tensors[n["distance"]].to(torch.float32)[rows].T)
         if self.row_norm:
             self.q_norm_w = tensors[n["q_norm"]]
             self.k_norm_w = None if self.kv_shared else tensors[n["k_norm"]]
@@ -362,10 +385,11 @@ class NormedAttention(Mixer):
         rotary = None if self.freq is None else (self.freq.data_ptr(), self.rot_dims, self.magnitude)
         return ("normed_attention", self.hidden, self.nh, self.nkv, self.dk, self.dv, self.scale, self.eps, self.values, self.taps,
                 self.has_gate, self.qk_norm, self.norm_weight, self.norm_where, self.q_temp, self.window, self.chunk, rotary,
-                self.gate_per_head, self.row_norm, self.has_bias, self.softcap, self.sink_kind, self.kv_shared)
+                self.gate_per_head, self.row_norm, self.has_bias, self.softcap, self.sink_kind, self.kv_shared, self.distance)
 
     def own_tensors(self):
-        return [self.w_in, self.w_o, self.q_norm_w, self.k_norm_w, self.w_conv, self.b_in, self.sink if self.sink_kind == "learned" else None]
+        return [self.w_in, self.w_o, self.q_norm_w, self.k_norm_w, self.w_conv, self.b_in, self.sink if self.sink_kind == "learned" else None,
+                self.bias.table if self.bias is not None else None]
 
     def _shared_kernels(self, page_size: int) -> bool:
         """Whether the attention itself runs on the kernels of equal key and value widths."""
@@ -415,25 +439,26 @@ class NormedAttention(Mixer):
             wide = o if (sv == self.dv and gate is None) else ctx.buffer("normed_attention.o_stored", (T, self.nh * sv), dt)
             attention_kernels.paged_attention(q, kv_view.pages, wide, ctx, kv_view.block_table, self.nh, self.nkv, sk, self.scale,
                                               self.window, beside_mma_products=gemm_bf16.gemv_preferred(x, self.w_o), chunk=self.chunk,
-                                              sink=self.sink, softcap=self.softcap or 0.0)
+                                              sink=self.sink, softcap=self.softcap or 0.0, bias=self.bias)
             if wide is not o:
                 attention_kv.gate_heads(wide, o, gate, self.conv_cols, self.nh, self.dv, sv, per_head=self.gate_per_head)
-        elif self.stored is not None and self.sink is None and not self.softcap:
+        elif self.stored is not None and self.sink is None and not self.softcap and self.bias is None:
             # a page size the tensor-core kernels do not take: the plain kernel of one width
             wide = ctx.buffer("normed_attention.o_stored", (T, self.nh * sv), dt)
             attention_kernels.paged_attention(q, kv_view.pages, wide, ctx, kv_view.block_table, self.nh, self.nkv, sk, self.scale, self.window,
                                               chunk=self.chunk)
             attention_kv.gate_heads(wide, o, gate, self.conv_cols, self.nh, self.dv, sv, per_head=self.gate_per_head)
         elif self.stored is not None:
-            # the same with a sink or a cap: the plain kernel of two widths, told that both are the stored one
+            # the same with a sink, a cap or a distance bias: the plain kernel of two widths, told that both are the stored one
             wide = ctx.buffer("normed_attention.o_stored", (T, self.nh * sv), dt)
             attention_kv.paged_attention_kv(q, kv_view.pages, wide, ctx.positions, ctx.token_seq, kv_view.block_table, kv_view.page_size,
                                             self.nh, self.nkv, sk, sv, self.scale, self.window, None, 0, flag, chunk=self.chunk,
-                                            sink=self.sink, softcap=self.softcap or 0.0)
+                                            sink=self.sink, softcap=self.softcap or 0.0, bias=self.bias)
             attention_kv.gate_heads(wide, o, gate, self.conv_cols, self.nh, self.dv, sv, per_head=self.gate_per_head)
         else:
             attention_kv.paged_attention_kv(q, kv_view.pages, o, ctx.positions, ctx.token_seq, kv_view.block_table, kv_view.page_size,
                                             self.nh, self.nkv, self.dk, self.dv, self.scale, self.window, gate, self.conv_cols, flag,
-                                            chunk=self.chunk, gate_per_head=self.gate_per_head, sink=self.sink, softcap=self.softcap or 0.0)
+                                            chunk=self.chunk, gate_per_head=self.gate_per_head, sink=self.sink, softcap=self.softcap or 0.0,
+                                            bias=self.bias)
         return linear(o, self.w_o, None, torch.float32, partials_ok=True, error_flag=flag,
                       alloc=lambda shape, dtype: ctx.buffer("normed_attention.out", shape, dtype))

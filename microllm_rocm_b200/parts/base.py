@@ -231,6 +231,11 @@ class Norm(Part):
         """residual += delta in place, then out = norm(residual)."""
         raise NotImplementedError
 
+    def fused_params(self):
+        """(weight, bias or None, eps, centred) when the norm is a plain layer norm (centred) or rms norm, for a kernel that
+        makes it as part of a larger step."""
+        raise NotImplementedError(f"{type(self).__name__} is not a norm that other kernels can make")
+
 
 @dataclass(frozen=True)
 class RotaryTable:

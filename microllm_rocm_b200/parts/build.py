@@ -55,6 +55,11 @@ class Model:
                              (feed_forward, layer.feed_forward)):
                 self._parts.append((layer.prefix + ps.params.get("prefix", ""), part))
             self._parts.append((layer.prefix + layer.block.params.get("prefix", ""), block))
+        for i, block in enumerate(self.blocks):
+            if getattr(block, "streams", None) != spec.streams:
+                raise ValueError(f"layer {i}: its block keeps {getattr(block, 'streams', None)} streams, the model {spec.streams}")
+        if spec.streams is not None and any(run.entry is not None for run in spec.order):
+            raise ValueError("run entries and several residual streams do not go together")
         # what a run does to the residual stream before its layer
         self.run_entries = []
         for run in spec.order:
@@ -137,8 +142,10 @@ class Model:
         return self._replay_keys
 
     @staticmethod
-    def _run_pointers(block, view) -> List[int]:
-        return [0 if t is None else t.data_ptr() for t in list(block.own_tensors()) + _view_tensors(view)]
+    def _run_pointers(block, view, delta) -> List[int]:
+        # (a pending delta may bring tensors of the layer before: they take part like the layer's own)
+        brought = delta.own_tensors() if hasattr(delta, "own_tensors") else []
+        return [0 if t is None else t.data_ptr() for t in list(block.own_tensors()) + _view_tensors(view) + brought]
 
     # --- weights ----------------------------------------------------------------------
     def expected_tensors(self) -> Dict[str, WeightSpec]:
@@ -214,8 +221,9 @@ class Model:
         self.position.on_embedding(residual, ctx)
         delta = None
         sink = ctx.tensor_sink
+        streams = self.spec.streams is not None
         if sink is not None:
-            sink("embedding", residual)
+            sink("embedding", residual[:, 0] if streams else residual)
         embedding_output = None
         if self._keep_embedding:                 # a later run adds the embedding output again: the residual is changed in place
             embedding_output = ctx.buffer("model.embedding_output", tuple(residual.shape), torch.float32)
@@ -241,11 +249,14 @@ class Model:
             if key is None:
                 # the first run of a step plans launches and makes the step's tables: it always runs call by call
                 residual, delta = block.forward(residual, delta, ctx, view)
-                if sink is not None:
+                if sink is not None and streams:                         # the sum of the streams, the pending result taken in
+                    sink(f"run{i}.layer{run.layer}.residual", block.total(residual, delta))
+                    sink(f"run{i}.layer{run.layer}.delta", None)
+                elif sink is not None:
                     sink(f"run{i}.layer{run.layer}.residual", residual)
                     sink(f"run{i}.layer{run.layer}.delta", delta)          # None where a block hands no delta on
                 continue
-            pointers = self._run_pointers(block, view)
+            pointers = self._run_pointers(block, view, delta)
             if key not in recordings:
                 from ..kernels.replay import Recorder, Recording
                 with Recorder() as recorder:
@@ -255,26 +266,31 @@ class Model:
                     out_delta is not None and delta is not None and out_delta.data_ptr() == delta.data_ptr())
                 if out_residual is residual and same_delta and recorder.unrecordable is None:
                     recording = Recording(recorder)
-                    if not _swappable(recording, block, view):
+                    if not _swappable(recording, block, view, delta):
                         recording = None
-                recordings[key] = (recording, pointers) if recording is not None else None
+                recordings[key] = (recording, pointers, out_delta) if recording is not None else None
                 residual, delta = out_residual, out_delta
                 continue
             entry = recordings[key]
-            if entry is None:
+            if entry is None or not _one_to_one(entry[1], pointers):
                 residual, delta = block.forward(residual, delta, ctx, view)
                 continue
-            recording, base = entry
+            recording, base, recorded_delta = entry
             recording.replay(list(zip(base, pointers)))
+            if hasattr(block, "pending"):            # a delta that names the layer's own tensors: the same buffer, this layer's
+                delta = block.pending(recorded_delta)
             self.layers_replayed += 1
         R = ctx.logit_rows.shape[0]
         if R == 0:
             return torch.empty((0, self.spec.vocab_size), dtype=torch.float32, device=residual.device)
-        if delta is not None:
-            from ..kernels import ops
-            ops.add_inplace(residual, delta)
         rows = torch.empty((R, self.spec.hidden_size), dtype=self.rt.dtype, device=residual.device)
-        self.final_norm.forward(residual, rows, rows=ctx.logit_rows)
+        if streams:
+            self.blocks[self.spec.order[-1].layer].final_forward(residual, delta, self.final_norm, rows, ctx.logit_rows)
+        else:
+            if delta is not None:
+                from ..kernels import ops
+                ops.add_inplace(residual, delta)
+            self.final_norm.forward(residual, rows, rows=ctx.logit_rows)
         logits = self.head.forward(rows, ctx.error_flag)
         if sink is not None:
             sink("final_norm", rows)
@@ -290,11 +306,19 @@ def _view_tensors(view) -> List[Optional[torch.Tensor]]:
     return [getattr(view, "pages", None), getattr(view, "storage", None)]
 
 
-def _swappable(recording, block, view) -> bool:
+def _one_to_one(base, pointers) -> bool:
+    """Whether every recorded address stands for one address of the run to be issued (a tensor that plays two parts in the
+    recorded run may play only one of them in another)."""
+    to = {}
+    return all(to.setdefault(a, b) == b for a, b in zip(base, pointers) if a)
+
+
+def _swappable(recording, block, view, delta=None) -> bool:
     """Every pointer a recorded launch takes into a tensor the layer owns must be that tensor's base address:
     only those can be replaced by another layer's tensor.  (A launcher handed `weight + offset` would keep
     reading the recorded layer's weight.)"""
-    owned = [t for t in list(block.own_tensors()) + _view_tensors(view) if t is not None]
+    brought = delta.own_tensors() if hasattr(delta, "own_tensors") else []
+    owned = [t for t in list(block.own_tensors()) + _view_tensors(view) + brought if t is not None]
     ranges = [(t.data_ptr(), t.data_ptr() + t.numel() * t.element_size()) for t in owned]
     for p in recording.pointers:
         for lo, hi in ranges:

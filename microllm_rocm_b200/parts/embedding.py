@@ -31,6 +31,10 @@ class TokenEmbedding(Part):
         if self.bigram and self.bigram["buckets"] <= 0:
             raise ValueError("token_embedding: bigram buckets must be positive")
         self.bigram_table: Optional[torch.Tensor] = None
+        # several residual streams: every token's row is written this many times, [T, streams, hidden] (None: one stream, [T, hidden])
+        self.streams = int(params["streams"]) if params.get("streams") else None
+        if self.streams and (self.norm or self.bigram):
+            raise ValueError("token_embedding: several streams with a norm or a pair table are not supported")
         self.rt = rt
         self.table: Optional[torch.Tensor] = None
 
@@ -48,7 +52,7 @@ class TokenEmbedding(Part):
         return specs
 
     def kernel_sources(self):
-        return [("residual.cu", {})] if self.scale != 1.0 or self.bigram else []
+        return [("residual.cu", {})] if self.scale != 1.0 or self.bigram or self.streams else []
 
     def bind(self, tensors):
         self.table = tensors[self.name]
@@ -59,6 +63,10 @@ class TokenEmbedding(Part):
 
     def forward(self, token_ids: torch.Tensor, ctx=None, state=None) -> torch.Tensor:
         """`ctx`, `state`: the step and the view of this part's per-sequence state; needed only with a pair table."""
+        if self.streams:
+            out = torch.empty((token_ids.shape[0], self.streams, self.hidden), dtype=torch.float32, device=token_ids.device)
+            ops.embed_gather_scaled(self.table, token_ids, out, self.scale)
+            return out
         out = torch.empty((token_ids.shape[0], self.hidden), dtype=torch.float32, device=token_ids.device)
         if self.bigram and (ctx is None or state is None):
             raise RuntimeError("token_embedding: a pair table needs the step's context and the sequences' state")

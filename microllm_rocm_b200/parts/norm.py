@@ -1,6 +1,6 @@
 """RMSNorm: y = x * (1 / sqrt(mean(x^2) + eps)) * w, all in fp32 (`one_plus`: the checkpoint stores w - 1, a weight around zero)
 (reference: src/ops/ops.cpp:684-699; fused with the residual add at :702-740).
-LayerNorm: y = (x - mean) / sqrt(mean((x - mean)^2) + eps) * w + b, all in fp32; besides the plain form it offers the
+LayerNorm: y = (x - mean) / sqrt(mean((x - mean)^2) + eps) * w + b, all in fp32 (`bias=False`: no b); besides the plain form it offers the
 step of a block that normalises AFTER its sums: x <- norm(alpha * x + weighted results), in place."""
 from __future__ import annotations
 
@@ -40,6 +40,10 @@ class RMSNorm(Norm):
     def own_tensors(self):
         return [self.weight]
 
+    def fused_params(self):
+        """(weight, bias, eps, centred) for a kernel that makes this norm as part of a larger step."""
+        return self.weight, None, self.eps, False
+
     def forward(self, x, out, rows=None):
         ops.rmsnorm(x, self.weight, self.eps, out, rows=rows)
 
@@ -58,7 +62,7 @@ class LayerNorm(Norm):
         self.size = int(params["size"])
         self.eps = float(params["eps"])
         self.name = params.get("name", "weight")
-        self.bias_name = params.get("bias_name", "bias")
+        self.bias_name = params.get("bias_name", "bias") if params.get("bias", True) else None
         self.absent = bool(params.get("absent", False))
         self.rt = rt
         self.weight: Optional[torch.Tensor] = None
@@ -67,22 +71,28 @@ class LayerNorm(Norm):
     def weight_specs(self) -> Dict[str, WeightSpec]:
         if self.absent:
             return {}
-        return {self.name: WeightSpec((self.size,), role="vector", init=("one_plus_normal", 0.1)),
-                self.bias_name: WeightSpec((self.size,), role="vector", init=("normal", 0.1))}
+        specs = {self.name: WeightSpec((self.size,), role="vector", init=("one_plus_normal", 0.1))}
+        if self.bias_name is not None:
+            specs[self.bias_name] = WeightSpec((self.size,), role="vector", init=("normal", 0.1))
+        return specs
 
     def kernel_sources(self):
         return [("layernorm.cu", {})]
 
     def bind(self, tensors):
-        self.weight, self.bias = tensors.get(self.name), tensors.get(self.bias_name)
-        if not self.absent and (self.weight is None or self.bias is None):
+        self.weight = tensors.get(self.name)
+        self.bias = tensors.get(self.bias_name) if self.bias_name is not None else None
+        if not self.absent and (self.weight is None or (self.bias is None and self.bias_name is not None)):
             raise KeyError(f"layer norm: {self.name} or {self.bias_name} is missing")
 
     def replay_key(self):
-        return ("layernorm", self.size, self.eps)
+        return ("layernorm", self.size, self.eps, self.bias_name is not None)
 
     def own_tensors(self):
         return [self.weight, self.bias]
+
+    def fused_params(self):
+        return self.weight, self.bias, self.eps, True
 
     def forward(self, x, out, rows=None):
         ops.layernorm(x, self.weight, self.bias, self.eps, out, rows=rows)

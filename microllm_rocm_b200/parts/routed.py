@@ -7,6 +7,10 @@
 
 `scoring="softmax_all"`: s = softmax(z) over ALL router outputs; the `top` largest s + correction are chosen (the correction,
 a tensor named by `router_bias_name`, only steers the choice) and the weights are the chosen s themselves, not renormalised.
+`scoring="sigmoid_groups"` with `groups`, `keep`, `weight_scale`: s = sigmoid(z); the experts form equal groups of neighbours, a
+group scores the sum of its two largest s, only experts of the `keep` best groups can be chosen; the weights are the chosen s
+divided by their sum, times `weight_scale`.  `activation="clamped_swish"` with `limit`: the experts' inner activation is the
+clamped form of the dense feed-forward.
 `identity` = n: the router has experts + n outputs, and the last n have no expert behind them: a token that chooses one gets
 its own input back, times the weight.
 
@@ -23,6 +27,7 @@ import torch
 
 from ..kernels import gemm_bf16, grouped, moe
 from ..kernels.linear import linear
+from ..kernels.ops import CLAMPED_ACTIVATION
 from .base import FEED_FORWARDS, FeedForward, Runtime, StepContext, WeightSpec, make, register_feed_forward, scratch
 
 
@@ -49,6 +54,18 @@ class RoutedExperts(FeedForward):
         self.identity = int(params.get("identity", 0))                 # router outputs behind the experts' that pass the input on
         if self.identity < 0:
             raise ValueError("routed experts: identity must not be negative")
+        self.groups, self.keep = int(params.get("groups", 1)), int(params.get("keep", 1))
+        self.weight_scale = float(params.get("weight_scale", 1.0))
+        if self.scoring == "sigmoid_groups":
+            if self.identity or self.groups <= 0 or self.experts % self.groups or not 0 < self.keep <= self.groups \
+                    or self.top > self.keep * (self.experts // self.groups):
+                raise ValueError(f"routed experts: top {self.top} of {self.keep} of {self.groups} groups of {self.experts} experts")
+        elif self.groups != 1 or self.weight_scale != 1.0:
+            raise ValueError(f"routed experts: scoring {self.scoring!r} has neither groups nor a factor on the weights")
+        self.activation = params.get("activation", "silu")
+        self.limit = float(params["limit"]) if params.get("limit") is not None else None
+        if self.activation not in ("silu", CLAMPED_ACTIVATION) or (self.activation == CLAMPED_ACTIVATION and not (self.limit or 0) > 0):
+            raise ValueError(f"routed experts: activation {self.activation!r} with limit {self.limit}")
         self.outputs = self.experts + self.identity                    # what the router chooses among
         self.shared = None
         self.shared_prefix = ""
@@ -133,7 +150,7 @@ class RoutedExperts(FeedForward):
         if not self.rt.is_fp32 and not gemm_bf16._direct_library(self.rt.device):
             return None                  # the library product would go through the tensor framework
         return ("routed_experts", self.hidden, self.experts, self.top, self.inter, shared, self.has_gate, self.b_router is not None,
-                self.scoring, self.identity)
+                self.scoring, self.identity, self.groups, self.keep, self.weight_scale, self.activation, self.limit)
 
     def own_tensors(self):
         own = [self.w_gate_up, self.w_down, self.w_router, self.b_router]
@@ -152,14 +169,15 @@ class RoutedExperts(FeedForward):
         # throughout); bias, choice, weights and the gate's sigmoid follow in fp32
         logits = linear(x, self.w_router, None, torch.float32, partials_ok=True, error_flag=flag,
                         alloc=lambda shape, dtype: buf("logits", shape, dtype))
-        moe.select(logits, self.outputs, self.b_router, top, ids, weights, self.outputs if self.has_gate else -1, gate, scoring=self.scoring)
+        moe.select(logits, self.outputs, self.b_router, top, ids, weights, self.outputs if self.has_gate else -1, gate, scoring=self.scoring,
+                   groups=self.groups, keep=self.keep, weight_scale=self.weight_scale)
         offsets = buf("offsets", (E + 1,), torch.int32)
         order = buf("order", (P,), torch.int32)
         moe.align(ids, E, offsets, order, flag, passthrough=self.identity)
         row_tile = grouped.row_tile_for(P, E, True, grouped.mma_supported(x, self.w_gate_up))
         act = buf("act", (P, ff), self.rt.dtype)
         grouped.grouped_silu_mul(x, self.w_gate_up, act, rows=P, group_offsets=offsets, a_rows=order, a_row_div=top,
-                                 row_tile=row_tile, alloc=lambda shape, dtype: buf("gate_up", shape, dtype))
+                                 row_tile=row_tile, alloc=lambda shape, dtype: buf("gate_up", shape, dtype), activation=self.activation, limit=self.limit)
         y = buf("y", (P, W), torch.float32)
         grouped.grouped_linear(act, self.w_down, y, rows=P, group_offsets=offsets, c_rows=order, row_tile=row_tile)
         shared = self.shared.forward(x, ctx) if self.shared is not None else None
