@@ -318,6 +318,12 @@ def step_timeline(session):
 # stand beside the closest design that was here before, a Fonuvik of the same width, layers and vocabulary: parallel layers
 # with the heads and widths of Lozepel's two sides where Lozepel has a softmax mixer, and routed experts of the same count
 # and width (plus a shared expert as wide as Lozepel's dense feed-forward where Lozepel has that).
+# The Gubidra sizes (several residual streams mixed around every sublayer; a layer of retention, one of the matrix memory with
+# exponential gates, two of windowed attention with a bias by distance and a gate per head; routed experts with a choice limited
+# to groups and a clamped activation in every layer) stand beside the closest design that was here before, a Lozepel of the
+# same width, layers and vocabulary: an attention layer with the same heads where Gubidra has one, a parallel layer (those
+# attention heads beside linear attention with the recurrence's heads and widths) where Gubidra has a recurrence, and routed
+# experts of the same count and width.
 DESIGN_SIZES = {
     "small": dict(gedalix="gedalix-small", layers=4),
     "16b-layers": dict(gedalix="gedalix-16b-layers", layers=4),
@@ -327,6 +333,8 @@ DESIGN_SIZES = {
     "fonuvik-3b-layers": dict(fonuvik="fonuvik-3b-layers", layers=4),
     "lozepel-small": dict(lozepel="lozepel-small", layers=4),
     "lozepel-3b-layers": dict(lozepel="lozepel-3b-layers", layers=4),
+    "gubidra-small": dict(gubidra="gubidra-small", layers=4),
+    "gubidra-3b-layers": dict(gubidra="gubidra-3b-layers", layers=4),
 }
 
 
@@ -384,6 +392,21 @@ def _equal_fonuvik_lozepel(raw, layers, max_positions):
                                     "layers": made, "max_positions": max_positions})
 
 
+def _equal_lozepel_gubidra(raw, layers, max_positions):
+    from microllm_rocm_b200.config.lozepel import LozepelConfig, attention_layer, moe, parallel_layer
+    soft = next(l["mixer"] for l in raw["layers"] if l["type"] == "attention")
+    made = []
+    for layer in raw["layers"][:layers]:
+        m, r = layer["mixer"], layer["mlp"]
+        ff = moe(r["router"]["experts"], r["router"]["top"], r["expert"]["ff"]) if r else None
+        if layer["type"] == "attention":
+            made.append(attention_layer(m["heads"], m["kv_heads"], m["dim"], ff, rot_dims=m["dim"]))
+        else:
+            made.append(parallel_layer(soft["heads"], soft["kv_heads"], soft["dim"], soft["vdim"], m["heads"], m["dim"], m["vdim"], ff))
+    return LozepelConfig.from_dict({"architecture": "Lozepel", "vocab": raw["vocab"], "width": raw["width"], "norm": {"eps": 1e-6},
+                                    "layers": made, "max_positions": max_positions})
+
+
 def _kernel_rows(step_fn, repeats=3):
     """(name, launches, summed duration in us, summed exposed time in us: see _exposed) of one call of step_fn, the
     kernels that add most to the step first.  Kernels start early behind their predecessors, so a duration holds
@@ -419,7 +442,13 @@ def run_designs(args):
     for name in names:
         size = DESIGN_SIZES[name]
         layers = args.layers or size["layers"]
-        if "lozepel" in size:
+        if "gubidra" in size:
+            from microllm_rocm_b200.config.gubidra import PRESETS as GUBIDRA_PRESETS, GubidraConfig
+            raw = copy.deepcopy(GUBIDRA_PRESETS[size["gubidra"]])
+            raw["layers"] = raw["layers"][:layers]
+            raw["max_positions"] = args.prompt + 512
+            designs = {"gubidra": GubidraConfig.from_dict(raw), "lozepel": _equal_lozepel_gubidra(raw, layers, args.prompt + 512)}
+        elif "lozepel" in size:
             from microllm_rocm_b200.config.lozepel import PRESETS as LOZEPEL_PRESETS, LozepelConfig
             raw = copy.deepcopy(LOZEPEL_PRESETS[size["lozepel"]])
             raw["layers"] = raw["layers"][:layers]

@@ -561,42 +561,72 @@ struct HeadPrepareParams {
     int* error_flag;
 };
 
-// One warp walks the tokens of one (sequence, head): the logs of 32 tokens' gates side by side in its lanes, the running
-// maximum from lane to lane, the exponentials side by side again.  The next 32 tokens' columns are fetched meanwhile.
-__device__ __forceinline__ void walk_gates(const HeadPrepareParams& p, int item) {
-    const int lane = threadIdx.x & 31, a = item / p.H, h = item % p.H;
+// A CTA walks the tokens of one (sequence, head) in chunks of GATE_CHUNK: every thread makes the logs of a token's two gates,
+// one thread carries the running maximum through the chunk, every thread makes a token's exponentials.  While that one
+// thread walks a chunk, the other warps finish the chunk before and prepare the one behind (the same thread reads a place
+// of the buffer and writes it anew).
+constexpr int GATE_CHUNK = 256;
+struct GateBuffers {
+    float2 log_gates[2][GATE_CHUNK];         // (f, i)
+    float m[2][GATE_CHUNK + 4];              // m[j]: the maximum in front of token j of the chunk
+};
+
+__device__ __forceinline__ void walk_gates(const HeadPrepareParams& p, int item, GateBuffers& s) {
+    const int a = item / p.H, h = item % p.H;
     const int start = p.seq_starts[a], n = p.seq_starts[a + 1] - start;
     const int slot = p.slots[a];
     if (slot < 0 || slot >= p.num_slots) {
-        if (lane == 0 && p.error_flag) atomicExch(p.error_flag, 3);
-        return;
+        if (threadIdx.x == 0 && p.error_flag) atomicExch(p.error_flag, 3);
+        return;                              // (the same for the whole CTA)
     }
-    float m = p.seq_pos0[a] == 0 ? 0.0f : p.m_state[(size_t)slot * p.H + h];
     const float bi = p.i_bias[h], bf = p.f_bias[h];
-    float ai = 0.0f, af = 0.0f;
-    if (lane < n) { ai = p.src.at(start + lane, p.i_col + h); af = p.src.at(start + lane, p.f_col + h); }
-    for (int base = 0; base < n; base += 32) {
-        const float i = p.cap * tanhf((ai + bi) / p.cap);
-        const float f = log_sigmoid(p.cap * tanhf((af + bf) / p.cap));
-        const int next = base + 32 + lane;
-        if (next < n) { ai = p.src.at(start + next, p.i_col + h); af = p.src.at(start + next, p.f_col + h); }
-        const int count = min(32, n - base);
-        float before = 0.0f, now = 0.0f;
+    auto prepare = [&](int chunk, int j) {
+        const int t = chunk * GATE_CHUNK + j;
+        if (t >= n) return;
+        const float i = p.cap * tanhf((p.src.at(start + t, p.i_col + h) + bi) / p.cap);
+        const float f = log_sigmoid(p.cap * tanhf((p.src.at(start + t, p.f_col + h) + bf) / p.cap));
+        s.log_gates[chunk & 1][j] = make_float2(f, i);
+    };
+    auto finish = [&](int chunk, int j) {
+        const int t = chunk * GATE_CHUNK + j;
+        if (t >= n) return;
+        const float2 g = s.log_gates[chunk & 1][j];
+        const float before = s.m[chunk & 1][j], now = s.m[chunk & 1][j + 1];
+        const size_t at = (size_t)(start + t) * p.H + h;
+        p.keep[at] = expf(g.x + before - now);
+        p.take[at] = expf(g.y - now);
+        p.floor[at] = expf(-now);
+    };
+    const int chunks = (n + GATE_CHUNK - 1) / GATE_CHUNK;
+    float m = p.seq_pos0[a] == 0 ? 0.0f : p.m_state[(size_t)slot * p.H + h];
+    for (int j = threadIdx.x; j < GATE_CHUNK; j += PREPARE_THREADS) prepare(0, j);
+    __syncthreads();
+    for (int c = 0; c < chunks; ++c) {
+        if (threadIdx.x == 0) {
+            const float2* g = s.log_gates[c & 1];
+            float* out = s.m[c & 1];
+            const int count = min(GATE_CHUNK, n - c * GATE_CHUNK);
+            out[0] = m;
+            int j = 0;
+            for (; j + 8 <= count; j += 8) {
+                float2 v[8];
 #pragma unroll
-        for (int j = 0; j < 32; ++j) {
-            const float fj = __shfl_sync(0xffffffffu, f, j), ij = __shfl_sync(0xffffffffu, i, j);
-            const float m_new = fmaxf(fj + m, ij);
-            if (lane == j) { before = m; now = m_new; }
-            if (j < count) m = m_new;
+                for (int k = 0; k < 8; ++k) v[k] = g[j + k];
+#pragma unroll
+                for (int k = 0; k < 8; ++k) { m = fmaxf(v[k].x + m, v[k].y); out[j + k + 1] = m; }
+            }
+            for (; j < count; ++j) { m = fmaxf(g[j].x + m, g[j].y); out[j + 1] = m; }
+        } else if (threadIdx.x >= 32) {
+            for (int j = threadIdx.x - 32; j < GATE_CHUNK; j += PREPARE_THREADS - 32) {
+                if (c > 0) finish(c - 1, j);
+                prepare(c + 1, j);
+            }
         }
-        if (lane < count) {
-            const size_t at = (size_t)(start + base + lane) * p.H + h;
-            p.keep[at] = expf(f + before - now);
-            p.take[at] = expf(i - now);
-            p.floor[at] = expf(-now);
-        }
+        __syncthreads();
     }
-    if (lane == 0) p.m_state[(size_t)slot * p.H + h] = m;
+    if (chunks > 0)
+        for (int j = threadIdx.x; j < GATE_CHUNK; j += PREPARE_THREADS) finish(chunks - 1, j);
+    if (threadIdx.x == 0) p.m_state[(size_t)slot * p.H + h] = m;
 }
 
 // what a column of q or k becomes: turned with its partner where it belongs to the turned part of its head, then scaled
@@ -615,8 +645,8 @@ template <bool FOUR>
 __global__ void __launch_bounds__(PREPARE_THREADS) head_decay_prepare_kernel(HeadPrepareParams p) {
     pdl_prologue();
     if ((int)blockIdx.x < p.gate_blocks) {                  // the serial part first: it takes longest
-        const int item = blockIdx.x * (PREPARE_THREADS / 32) + (threadIdx.x >> 5);
-        if (item < p.A * p.H) walk_gates(p, item);
+        __shared__ GateBuffers buffers;
+        walk_gates(p, blockIdx.x, buffers);
         return;
     }
     constexpr int N = FOUR ? 4 : 1;
@@ -667,10 +697,9 @@ MLB_EXPORT int mlb_head_decay_prepare(const float* src, long long ld, int n_part
     if (i_bias && (!f_bias || !m_state || !slots || !seq_starts || !seq_pos0 || !gates || !(cap > 0.0f)))
         return fail(MLB_INVALID_ARGUMENT, "head_decay_prepare: the gates need biases, a cap, a state and the step's sequences");
     if (T == 0) return MLB_OK;
-    const int warps = PREPARE_THREADS / 32;
     const size_t plane = (size_t)T * H;
     HeadPrepareParams p{Columns{src, ld, n_partials, partial_stride}, q_col, k_col, v_col, (const float2*)cos_sin, rot_dims, q_scale, k_scale,
-                        q_out, k_out, v_out, T, H, DK, DV, i_bias ? (A * H + warps - 1) / warps : 0, i_col, f_col, i_bias, f_bias, cap,
+                        q_out, k_out, v_out, T, H, DK, DV, i_bias ? A * H : 0, i_col, f_col, i_bias, f_bias, cap,
                         m_state, slots, num_slots, seq_starts, seq_pos0, A, gates, gates ? gates + plane : nullptr,
                         gates ? gates + 2 * plane : nullptr, error_flag};
     const long long n = (long long)T * (2LL * H * DK + (long long)H * DV);
