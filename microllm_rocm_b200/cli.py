@@ -85,6 +85,8 @@ class TensorTrace:
 
     def __call__(self, name, tensor) -> None:
         import torch
+        if tensor is None:               # the delta of a block that hands none on
+            return
         values = tensor.detach().to(torch.float64).reshape(-1).cpu()
         finite = values[torch.isfinite(values)]
         stats = {"numel": int(values.numel()), "finite_count": int(finite.numel()), "minimum": 0.0, "maximum": 0.0,

@@ -1,4 +1,6 @@
 """The command line's flag rules, which follow the reference's (apps/hf_infer.cpp:179-285): no GPU needed."""
+import json
+
 import pytest
 
 from microllm_rocm_b200 import cli
@@ -71,3 +73,17 @@ def test_help_lists_every_option(capsys):
     text = capsys.readouterr().out
     for name in cli.DEFAULTS:
         assert f"--{name} " in text
+
+
+def test_tensor_trace_skips_what_a_block_does_not_hand_on(tmp_path):
+    import torch
+
+    from microllm_rocm_b200.cli import TensorTrace
+    trace = TensorTrace(str(tmp_path / "t" / "trace.jsonl"), 2, "float32")
+    trace("run0.layer0.residual", torch.tensor([[1.0, 2.0, float("nan")]]))
+    trace("run0.layer0.delta", None)
+    trace("logits", torch.ones(1, 3))
+    assert trace.write() == 2
+    records = [json.loads(line) for line in open(tmp_path / "t" / "trace.jsonl")]
+    assert [(r["name"], r["sequence"], r["shape"]) for r in records] == [("run0.layer0.residual", 0, [1, 3]), ("logits", 1, [1, 3])]
+    assert records[0]["statistics"]["finite_count"] == 2 and records[0]["values"] == [1.0, 2.0]
