@@ -9,7 +9,7 @@ What is held when:
   * `commit(request, new_len)` records the new length after a step ran, and gives back the
     pages of windowed groups that no later query can reach: a query at position p reads keys
     >= p - W + 1, so once the request holds n tokens, blocks that end at or before n - W + 1
-    are dead.
+    are dead -- except those that hold one of the group's first `keep_first` tokens, which stay visible.
   * `release(request)` gives back everything the request holds, pages and state slot.
 Freed pages are not cleared; a key is valid because of the request's length, not because of
 what the page holds.
@@ -34,7 +34,15 @@ GUARD_VALUE = -24576.0     # exact in bf16 and fp32; what a guard page holds
 
 
 def group_key(need) -> str:
-    return "full" if need.window is None else f"window{int(need.window)}"
+    if need.window is None:
+        return "full"
+    keep = kept_tokens(need)
+    return f"window{int(need.window)}" + (f"+{keep}" if keep else "")
+
+
+def kept_tokens(need) -> int:
+    """First tokens of a request that a windowed entry keeps for good."""
+    return int(getattr(need, "keep_first", 0) or 0) if need.window is not None else 0
 
 
 def page_shape(need, page_size: int):
@@ -55,8 +63,8 @@ class _Request:
 
 
 class CacheGroup:
-    def __init__(self, key: str, window: Optional[int], num_pages: int):
-        self.key, self.window = key, window
+    def __init__(self, key: str, window: Optional[int], num_pages: int, keep_first: int = 0):
+        self.key, self.window, self.keep_first = key, window, keep_first
         self.pool = PagePool(num_pages)
 
 
@@ -67,8 +75,8 @@ class CacheManager:
         """entries: cache name -> PagedKVNeed | FixedStateNeed (from parts.Model.cache_entries).
         num_pages: pages of a group that keeps all keys.  device None: books only, no storage (for host tests).
         max_step_tokens: the most tokens one request brings in a step, when the caller promises one: a group
-        with a window of W keys then never holds more than W - 1 + max_step_tokens tokens of a request, and its
-        pool (and storage) is sized for max_requests such spans instead of for num_pages.
+        with a window of W keys then never holds more than W - 1 + max_step_tokens tokens of a request (and the first
+        tokens it keeps), and its pool (and storage) is sized for max_requests such spans instead of for num_pages.
         guard_pages: a debugging aid.  Every paged entry's storage gets one more page in front and one behind,
         filled with a fixed pattern that no kernel may touch; check_guards() reads them back.  A store that runs off
         either end of the pool (a page index of -1 or num_pages that slipped through a kernel's checks) shows there."""
@@ -87,7 +95,7 @@ class CacheManager:
             if isinstance(need, (PagedKVNeed, PagedRowsNeed)):
                 key = group_key(need)
                 if key not in self.groups:
-                    self.groups[key] = CacheGroup(key, need.window, self.pages_for_group(need.window, max_step_tokens))
+                    self.groups[key] = CacheGroup(key, need.window, self.pages_for_group(need.window, max_step_tokens, kept_tokens(need)), kept_tokens(need))
                 self.entry_group[name] = key
                 if device is not None:
                     pages = self.groups[key].pool.num_pages + 1        # the pool's pages, then the spare page (see pad_page)
@@ -115,13 +123,13 @@ class CacheManager:
         self.pages_released_by_window = 0
         self.tables_version = 0          # grows whenever any block table changes: lets a reader skip a comparison
 
-    def pages_for_group(self, window: Optional[int], max_step_tokens: Optional[int]) -> int:
+    def pages_for_group(self, window: Optional[int], max_step_tokens: Optional[int], keep_first: int = 0) -> int:
         """Pages of a group's pool: num_pages for all keys; for a window, what max_requests requests can hold at
         most while each keeps W - 1 old keys and brings up to max_step_tokens new ones (one more block for a span
-        that does not start on a block's edge) -- never more than num_pages."""
+        that does not start on a block's edge) beside the blocks of the first tokens that stay -- never more than num_pages."""
         if window is None or not max_step_tokens:
             return self.num_pages
-        span_blocks = self.blocks_for(int(window) - 1 + int(max_step_tokens)) + 1
+        span_blocks = self.blocks_for(int(window) - 1 + int(max_step_tokens)) + 1 + self.blocks_for(keep_first)
         return max(1, min(self.num_pages, self.max_requests * span_blocks))
 
     # ----- requests -------------------------------------------------------------------------
@@ -189,7 +197,7 @@ class CacheManager:
                 continue
             first_needed = new_len - window + 1          # the next query, at position new_len, reads from here
             dead_blocks = max(0, first_needed) // self.page_size     # blocks wholly before first_needed
-            for b in range(min(dead_blocks, len(table))):
+            for b in range(self.blocks_for(self.groups[k].keep_first), min(dead_blocks, len(table))):
                 if table[b] != RELEASED:
                     self.groups[k].pool.free(table[b])
                     table[b] = RELEASED

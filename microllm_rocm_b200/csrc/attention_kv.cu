@@ -13,7 +13,8 @@
 //                           32 at absolute multiples of 32 with a running maximum and sum (the order of every addition
 //                           depends on the position alone, not on how the tokens were cut into steps), optional window,
 //                           optional output gate: o * sigmoid(gate) with the gate read from a projection's fp32 output
-//                           (one gate per element of a head, or one per head); optional bias per head and distance
+//                           (one gate per element of a head, or one per head); optional first tokens that stay visible in
+//                           front of the window; optional bias per head and distance
 //                           query - key, added to the scaled score; optional cap on the scores,
 //                           s <- cap * tanh(s / cap); optional sink: exp(sink[head]) joins the softmax's denominator
 //                           (no key, no value, neither scaled nor capped).
@@ -151,6 +152,7 @@ struct AttnParams {
     int tokens, num_heads, num_kv_heads, dk, dv;
     int chunk;               // > 0: only keys of the query's own block of `chunk` positions (counted from 0)
     int window;              // 0: all earlier keys
+    int keep;                // the first `keep` tokens stay visible in front of the window
     float scale;
     Columns gate; int gate_col;      // gate.base null: no gate
     int gate_per_head;               // 1: one gate per (token, head) at gate_col + head; 0: one per element at gate_col + head * dv + c
@@ -189,9 +191,10 @@ __global__ void __launch_bounds__(WARPS * 32) paged_attention_kv_kernel(AttnPara
     const int* table = p.block_table + (size_t)seq * p.max_blocks;
 
     const float* const bias_row = p.bias.table ? p.bias.row(h) : nullptr;
-    for (int base = (lo / 32) * 32; base <= pos; base += 32) {
-        const int kp = base + lane;
-        bool valid = kp >= lo && kp <= pos;
+    const KeyTiles tiles = key_tiles(lo, pos, p.keep, 32);
+    for (int i = 0; i < tiles.count; ++i) {
+        const int kp = tiles.at(i) * 32 + lane;
+        bool valid = key_visible(kp, pos, lo, p.keep);
         long long k_off = -1, v_off = -1;
         if (valid) {
             const int block = kp / p.page_size;
@@ -412,18 +415,18 @@ MLB_EXPORT int mlb_qk_prepare(const float* src, long long ld, int n_partials, lo
 MLB_EXPORT int mlb_paged_attention_kv(const void* q, int q_dtype, const void* pages, int kv_dtype, void* out, int out_dtype,
                                       const int* positions, const int* token_seq, const int* block_table, int max_blocks,
                                       int num_pages, int page_size, int tokens, int num_heads, int num_kv_heads, int dk, int dv,
-                                      int window, int chunk, float scale, const float* gate, long long gate_ld, int gate_partials,
+                                      int window, int keep, int chunk, float scale, const float* gate, long long gate_ld, int gate_partials,
                                       long long gate_partial_stride, int gate_col, int gate_per_head, const float* sink, float softcap,
                                       const float* distance_bias, int last_distance, int* error_flag, cudaStream_t stream) {
     if (tokens < 0 || num_heads <= 0 || num_kv_heads <= 0 || num_heads % num_kv_heads != 0)
         return fail(MLB_INVALID_ARGUMENT, "paged_attention_kv: bad head counts %d/%d", num_heads, num_kv_heads);
     if (dk <= 0 || dk > MAX_D || dv <= 0 || dv > MAX_D)
         return fail(MLB_UNSUPPORTED_SIZE, "paged_attention_kv: widths %d/%d not in 1..%d", dk, dv, MAX_D);
-    if (page_size <= 0 || num_pages <= 0 || max_blocks <= 0 || window < 0 || chunk < 0)
+    if (page_size <= 0 || num_pages <= 0 || max_blocks <= 0 || window < 0 || chunk < 0 || keep < 0)
         return fail(MLB_INVALID_ARGUMENT, "paged_attention_kv: bad cache geometry");
     if (tokens == 0) return MLB_OK;
     AttnParams p{q, pages, out, positions, token_seq, block_table, max_blocks, num_pages, page_size, tokens, num_heads,
-                 num_kv_heads, dk, dv, chunk, window, scale, Columns{gate, gate_ld, gate_partials < 1 ? 1 : gate_partials, gate_partial_stride},
+                 num_kv_heads, dk, dv, chunk, window, keep, scale, Columns{gate, gate_ld, gate_partials < 1 ? 1 : gate_partials, gate_partial_stride},
                  gate_col, gate_per_head ? 1 : 0, sink, softcap, DistanceBias{distance_bias, last_distance}, error_flag};
     if (distance_bias && last_distance < 0) return fail(MLB_INVALID_ARGUMENT, "paged_attention_kv: a distance bias has a last distance");
     if (softcap < 0.0f) return fail(MLB_INVALID_ARGUMENT, "paged_attention_kv: a cap on the scores is positive (0: none)");

@@ -62,6 +62,7 @@ struct FaParams {
     int num_heads, num_kv_heads, group;
     int chunk;               // > 0: only keys of the query's own block of `chunk` positions (counted from 0)
     int window;
+    int keep;                // the first `keep` tokens of a sequence stay visible in front of the window
     float scale_log2;               // softmax scale * log2(e); with a cap on the scores: cap * log2(e)
     int page_shift;                 // log2(page_size) when it is a power of two, else -1
     int* error_flag;
@@ -241,7 +242,7 @@ __device__ __forceinline__ void consume_keys(const FaParams& p, const __nv_bfloa
     }
     // Masks only where the tile touches an edge (the newest key, the window's start); a padding row
     // (position -1) of an interior tile keeps finite scores that are never stored.
-    const bool edge = kv.base + 15 > first_pos || kv.base < last_lo;           // uniform over the warp
+    const bool edge = kv.base + 15 > first_pos || (kv.base < last_lo && kv.base + 16 > p.keep);           // uniform over the warp
     float mx[2] = {-INFINITY, -INFINITY};
     if (edge) {
 #pragma unroll
@@ -250,7 +251,7 @@ __device__ __forceinline__ void consume_keys(const FaParams& p, const __nv_bfloa
             for (int e = 0; e < 4; ++e) {
                 const int i = e >> 1;
                 const int key = kv.base + nb * 8 + 2 * t + (e & 1);
-                const bool ok = key >= lo_row[i] && key <= pos_row[i];
+                const bool ok = key_visible(key, pos_row[i], lo_row[i], p.keep);
                 s[nb][e] = ok ? score_log2(p, s[nb][e], bias_row[i], pos_row[i] - key) : -INFINITY;
                 mx[i] = fmaxf(mx[i], s[nb][e]);
             }
@@ -321,13 +322,13 @@ __device__ __forceinline__ void consume_keys(const FaParams& p, const __nv_bfloa
     }
 }
 
-// Keys [tile_begin, tile_end) in units of 16, visiting every `stride`-th starting at
+// Key tiles number [tile_begin, tile_end) of the list `tiles` (16 keys each), visiting every `stride`-th starting at
 // tile_begin + first.  `a` and `b` are the register homes of the first and second tile; the caller
 // has already issued the loads of the first `in_flight` of them (b only where PREFETCH).  q_s: this tile's queries, [16][Q_STRIDE] bf16 in shared memory.  With
 // PREFETCH the loads of the next key tile are in flight while the current one is consumed.
 template <bool PREFETCH>
 __device__ __forceinline__ void attend(const FaParams& p, const TileGeometry& geo, const PageTable& pt,
-                                       const __nv_bfloat16* q_s, int tile_begin, int tile_end, int first, int stride,
+                                       const __nv_bfloat16* q_s, const KeyTiles& tiles, int tile_begin, int tile_end, int first, int stride,
                                        int hi_tile, RowState& st, KeyTile& a, KeyTile& b, int in_flight) {
     const int lane = threadIdx.x & 31, g = lane >> 2;
     int pos_row[2], lo_row[2];
@@ -357,23 +358,23 @@ __device__ __forceinline__ void attend(const FaParams& p, const TileGeometry& ge
     int kt = tile_begin + first;
     if (kt >= tile_end) return;
     if (PREFETCH) {
-        if (in_flight < 1) load_keys(p, geo, pt, kt, hi_tile, a);
+        if (in_flight < 1) load_keys(p, geo, pt, tiles.at(kt), hi_tile, a);
         while (true) {
             const bool more_b = kt + stride < tile_end;
-            if (more_b && in_flight < 2) load_keys(p, geo, pt, kt + stride, hi_tile, b);
+            if (more_b && in_flight < 2) load_keys(p, geo, pt, tiles.at(kt + stride), hi_tile, b);
             in_flight = 0;
             consume_keys(p, q_s, a, pos_row, lo_row, bias_row, first_pos, last_lo, st);
             if (!more_b) break;
             kt += stride;
             const bool more_a = kt + stride < tile_end;
-            if (more_a) load_keys(p, geo, pt, kt + stride, hi_tile, a);
+            if (more_a) load_keys(p, geo, pt, tiles.at(kt + stride), hi_tile, a);
             consume_keys(p, q_s, b, pos_row, lo_row, bias_row, first_pos, last_lo, st);
             if (!more_a) break;
             kt += stride;
         }
     } else {
         for (; kt < tile_end; kt += stride) {
-            if (in_flight < 1) load_keys(p, geo, pt, kt, hi_tile, a);
+            if (in_flight < 1) load_keys(p, geo, pt, tiles.at(kt), hi_tile, a);
             in_flight = 0;
             consume_keys(p, q_s, a, pos_row, lo_row, bias_row, first_pos, last_lo, st);
         }
@@ -429,7 +430,7 @@ __device__ __forceinline__ void ldmatrix_x4_trans(unsigned (&r)[4], const __nv_b
 constexpr int SWZ_MASK = CHUNKS >= 8 ? 7 : CHUNKS - 1;
 __device__ __forceinline__ int swz(int key, int chunk) { return key * D + ((chunk ^ (key & SWZ_MASK)) << 3); }
 
-// Copy keys [base, base + 64) of (sequence, kv head) into one stage.  Keys outside [lo, hi] --
+// Copy keys [base, base + 64) of (sequence, kv head) into one stage.  Keys that no row sees --
 // behind every row's window (their pages may have been given back) or never written by this
 // sequence -- become zeros; a key inside the range without a page raises the error flag.
 // Thread `tid` always moves chunk tid % CHUNKS of keys tid / CHUNKS + j * KEYS_PER_PASS.
@@ -447,7 +448,7 @@ __device__ __forceinline__ void load_kv_stage(const FaParams& p, const PageTable
     for (int j = 0; j < PASSES; ++j) {
         const int key = key0 + j * KEYS_PER_PASS;
         const int pos = base + key;
-        const bool wanted = pos >= lo && pos <= hi;
+        const bool wanted = key_visible(pos, hi, lo, p.keep);
         const int page = wanted ? pt.page_of(pos / p.page_size) : -1;
         const bool ok = page >= 0 && page < p.num_pages;
         if (!ok && wanted && p.error_flag) atomicExch(p.error_flag, 3);
@@ -483,7 +484,7 @@ __global__ void __launch_bounds__(WARPS * 32, 2) fa_prefill_kernel(FaParams p) {
     const int cta_row_first = first_tile * 16, cta_row_last = min(total_rows, cta_row_first + WARPS * 16) - 1;
     const int cta_first_pos = geo.pos0 + cta_row_first / p.group, cta_last_pos = geo.pos0 + cta_row_last / p.group;
     const int cta_lo = first_visible_key(cta_first_pos, p.window, p.chunk);
-    const int tile_first = cta_lo / KEY_TILE, tile_last = cta_last_pos / KEY_TILE;
+    const KeyTiles tiles = key_tiles(cta_lo, cta_last_pos, p.keep, KEY_TILE);
 
     PageTable pt;
     {
@@ -507,7 +508,7 @@ __global__ void __launch_bounds__(WARPS * 32, 2) fa_prefill_kernel(FaParams p) {
         *reinterpret_cast<uint4*>(my_q + r * QO_STRIDE + c) = v;
     }
     __syncthreads();                                   // table and queries are in place
-    load_kv_stage(p, pt, geo.kvh, tile_first * KEY_TILE, cta_lo, cta_last_pos, kv_s);
+    load_kv_stage(p, pt, geo.kvh, tiles.at(0) * KEY_TILE, cta_lo, cta_last_pos, kv_s);
 
     // this thread's two rows
     int pos_row[2], lo_row[2];
@@ -549,17 +550,17 @@ __global__ void __launch_bounds__(WARPS * 32, 2) fa_prefill_kernel(FaParams p) {
         for (int e = 0; e < 4; ++e) o[nb][e] = 0.0f;
     float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.0f, 0.0f};
 
-    for (int kt = tile_first; kt <= tile_last; ++kt) {
-        const int stage = (kt - tile_first) & 1;
-        if (kt < tile_last) {
-            load_kv_stage(p, pt, geo.kvh, (kt + 1) * KEY_TILE, cta_lo, cta_last_pos, kv_s + (stage ^ 1) * KV_STAGE_ELEMS);
+    for (int kt = 0; kt < tiles.count; ++kt) {
+        const int stage = kt & 1;
+        if (kt + 1 < tiles.count) {
+            load_kv_stage(p, pt, geo.kvh, tiles.at(kt + 1) * KEY_TILE, cta_lo, cta_last_pos, kv_s + (stage ^ 1) * KV_STAGE_ELEMS);
             asm volatile("cp.async.wait_group 1;" ::: "memory");
         } else {
             asm volatile("cp.async.wait_group 0;" ::: "memory");
         }
         __syncthreads();
-        const int base = kt * KEY_TILE;
-        if (active && base <= warp_last_pos && base + KEY_TILE - 1 >= warp_lo) {
+        const int base = tiles.at(kt) * KEY_TILE;
+        if (active && base <= warp_last_pos && (base + KEY_TILE - 1 >= warp_lo || base < p.keep)) {
             const __nv_bfloat16* k_s = kv_s + stage * KV_STAGE_ELEMS;
             const __nv_bfloat16* v_s = k_s + KEY_TILE * D;
             // ---- S = Q K^T : 8 key blocks of 8 --------------------------------------------------
@@ -582,7 +583,7 @@ __global__ void __launch_bounds__(WARPS * 32, 2) fa_prefill_kernel(FaParams p) {
             // ---- masks and the running softmax ----------------------------------------------------
             float mx[2] = {-INFINITY, -INFINITY};
             // a tile that lies inside every row's range (all 16 rows exist) needs no mask
-            const bool interior = base + KEY_TILE - 1 <= warp_first_pos && base >= warp_lo_last && warp_rows_full;
+            const bool interior = base + KEY_TILE - 1 <= warp_first_pos && (base >= warp_lo_last || base + KEY_TILE <= p.keep) && warp_rows_full;
             if (interior) {
 #pragma unroll
                 for (int nb = 0; nb < 8; ++nb)
@@ -598,7 +599,7 @@ __global__ void __launch_bounds__(WARPS * 32, 2) fa_prefill_kernel(FaParams p) {
                     for (int e = 0; e < 4; ++e) {
                         const int i = e >> 1;
                         const int key = base + nb * 8 + 2 * t + (e & 1);
-                        const bool ok = key >= lo_row[i] && key <= pos_row[i];
+                        const bool ok = key_visible(key, pos_row[i], lo_row[i], p.keep);
                         s[nb][e] = ok ? score_log2(p, s[nb][e], bias_row[i], pos_row[i] - key) : -INFINITY;
                         mx[i] = fmaxf(mx[i], s[nb][e]);
                     }
@@ -732,7 +733,8 @@ __global__ void __launch_bounds__(DW * 32, DW == 4 ? 2 : 1) fa_decode_kernel(FaP
     geo.pos0 = pos0_load;
     const int last_pos = geo.pos0;
     const int lo = first_visible_key(last_pos, p.window, p.chunk);
-    int tile_begin = lo / 16, tile_end = last_pos / 16 + 1;
+    const KeyTiles tiles = key_tiles(lo, last_pos, p.keep, 16);
+    int tile_begin = 0, tile_end = tiles.count;
     const int splits = (int)gridDim.z, rank = (int)blockIdx.z;
     if (splits > 1) {                        // this CTA's even share of the sequence's key tiles
         const int per_split = (tile_end - tile_begin + splits - 1) / splits;
@@ -745,11 +747,11 @@ __global__ void __launch_bounds__(DW * 32, DW == 4 ? 2 : 1) fa_decode_kernel(FaP
     KeyTile tile_a, tile_b;
     const int first_kt = tile_begin + warp;
     int early = 0;
-    if (first_kt < tile_end && first_kt < last_pos / 16) {
-        load_keys(p, geo, pt, first_kt, last_pos, tile_a);
+    if (first_kt < tile_end && tiles.at(first_kt) < last_pos / 16) {
+        load_keys(p, geo, pt, tiles.at(first_kt), last_pos, tile_a);
         early = 1;
-        if (USE_PREFETCH && first_kt + DW < tile_end && first_kt + DW < last_pos / 16) {
-            load_keys(p, geo, pt, first_kt + DW, last_pos, tile_b);
+        if (USE_PREFETCH && first_kt + DW < tile_end && tiles.at(first_kt + DW) < last_pos / 16) {
+            load_keys(p, geo, pt, tiles.at(first_kt + DW), last_pos, tile_b);
             early = 2;
         }
     }
@@ -769,7 +771,7 @@ __global__ void __launch_bounds__(DW * 32, DW == 4 ? 2 : 1) fa_decode_kernel(FaP
     __syncthreads();
     RowState st;
     init_state(st);
-    attend<USE_PREFETCH>(p, geo, pt, q_s, tile_begin, tile_end, warp, DW, last_pos, st, tile_a, tile_b, early);
+    attend<USE_PREFETCH>(p, geo, pt, q_s, tiles, tile_begin, tile_end, warp, DW, last_pos, st, tile_a, tile_b, early);
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
         st.l[i] += __shfl_xor_sync(0xffffffffu, st.l[i], 1);
@@ -889,10 +891,10 @@ __device__ __forceinline__ void consume_keys_t(const FaParams& p, const __nv_bfl
     float s[4];
 #pragma unroll
     for (int e = 0; e < 4; ++e) s[e] = score_log2(p, s0[e] + s1[e], bias_row[e & 1], last_pos - (kv.base + g + 8 * (e >> 1)));
-    if (kv.base + 15 > last_pos || kv.base < lo) {         // an edge tile (uniform over the warp)
+    if (kv.base + 15 > last_pos || (kv.base < lo && kv.base + 16 > p.keep)) {         // an edge tile (uniform over the warp)
         const int key0 = kv.base + g, key1 = key0 + 8;
-        if (key0 < lo || key0 > last_pos) s[0] = s[1] = -INFINITY;
-        if (key1 < lo || key1 > last_pos) s[2] = s[3] = -INFINITY;
+        if (!key_visible(key0, last_pos, lo, p.keep)) s[0] = s[1] = -INFINITY;
+        if (!key_visible(key1, last_pos, lo, p.keep)) s[2] = s[3] = -INFINITY;
     }
     float mx[2] = {fmaxf(s[0], s[2]), fmaxf(s[1], s[3])};
     float corr[2];
@@ -1084,7 +1086,8 @@ __global__ void __launch_bounds__(DW * 32, DW == 4 ? 2 : 1) fa_decode_t_kernel(F
     geo.pos0 = pos0_load;
     const int last_pos = geo.pos0;
     const int lo = first_visible_key(last_pos, p.window, p.chunk);
-    int tile_begin = lo / 16, tile_end = last_pos / 16 + 1;
+    const KeyTiles tiles = key_tiles(lo, last_pos, p.keep, 16);
+    int tile_begin = 0, tile_end = tiles.count;
     const int splits = (int)gridDim.z, rank = (int)blockIdx.z;
     if (splits > 1) {                        // this CTA's even share of the sequence's key tiles
         const int per_split = (tile_end - tile_begin + splits - 1) / splits;
@@ -1096,11 +1099,11 @@ __global__ void __launch_bounds__(DW * 32, DW == 4 ? 2 : 1) fa_decode_t_kernel(F
     KeyTile tile_a, tile_b;
     int kt = tile_begin + warp;
     int in_flight = 0;
-    if (kt < tile_end && kt < last_pos / 16) {
-        load_keys(p, geo, pt, kt, last_pos, tile_a);
+    if (kt < tile_end && tiles.at(kt) < last_pos / 16) {
+        load_keys(p, geo, pt, tiles.at(kt), last_pos, tile_a);
         in_flight = 1;
-        if (USE_PREFETCH && kt + DW < tile_end && kt + DW < last_pos / 16) {
-            load_keys(p, geo, pt, kt + DW, last_pos, tile_b);
+        if (USE_PREFETCH && kt + DW < tile_end && tiles.at(kt + DW) < last_pos / 16) {
+            load_keys(p, geo, pt, tiles.at(kt + DW), last_pos, tile_b);
             in_flight = 2;
         }
     }
@@ -1126,23 +1129,23 @@ __global__ void __launch_bounds__(DW * 32, DW == 4 ? 2 : 1) fa_decode_t_kernel(F
     bias_rows_t(p, geo.kvh, bias_row);
     if (kt < tile_end) {
         if (USE_PREFETCH) {
-            if (in_flight < 1) load_keys(p, geo, pt, kt, last_pos, tile_a);
+            if (in_flight < 1) load_keys(p, geo, pt, tiles.at(kt), last_pos, tile_a);
             while (true) {
                 const bool more_b = kt + DW < tile_end;
-                if (more_b && in_flight < 2) load_keys(p, geo, pt, kt + DW, last_pos, tile_b);
+                if (more_b && in_flight < 2) load_keys(p, geo, pt, tiles.at(kt + DW), last_pos, tile_b);
                 in_flight = 0;
                 consume_keys_t(p, q_s, tile_a, last_pos, lo, bias_row, st);
                 if (!more_b) break;
                 kt += DW;
                 const bool more_a = kt + DW < tile_end;
-                if (more_a) load_keys(p, geo, pt, kt + DW, last_pos, tile_a);
+                if (more_a) load_keys(p, geo, pt, tiles.at(kt + DW), last_pos, tile_a);
                 consume_keys_t(p, q_s, tile_b, last_pos, lo, bias_row, st);
                 if (!more_a) break;
                 kt += DW;
             }
         } else {
             for (; kt < tile_end; kt += DW) {
-                if (in_flight < 1) load_keys(p, geo, pt, kt, last_pos, tile_a);
+                if (in_flight < 1) load_keys(p, geo, pt, tiles.at(kt), last_pos, tile_a);
                 in_flight = 0;
                 consume_keys_t(p, q_s, tile_a, last_pos, lo, bias_row, st);
             }
@@ -1266,7 +1269,8 @@ __global__ void __launch_bounds__(160, 2) fa_decode_ring_kernel(const __grid_con
     geo.pos0 = pos0_load;
     const int last_pos = geo.pos0;
     const int lo = first_visible_key(last_pos, p.window, p.chunk);
-    int tile_begin = lo / 16, tile_end = last_pos / 16 + 1;
+    const KeyTiles tiles = key_tiles(lo, last_pos, p.keep, 16);
+    int tile_begin = 0, tile_end = tiles.count;
     const int splits = (int)gridDim.z, rank = (int)blockIdx.z;
     if (splits > 1) {                        // this CTA's even share of the sequence's key tiles
         const int per_split = (tile_end - tile_begin + splits - 1) / splits;
@@ -1298,14 +1302,14 @@ __global__ void __launch_bounds__(160, 2) fa_decode_ring_kernel(const __grid_con
                 const int kt0 = tile_begin + 4 * i, n_tiles = min(4, tile_end - kt0);
                 // the tile that holds the new token's key was written by the kernel in front: everything before it
                 // travels while that kernel still runs
-                if (!waited && kt0 + n_tiles > last_pos / 16) { pdl_wait(); waited = true; }
+                if (!waited && tiles.at(kt0 + n_tiles - 1) >= last_pos / 16) { pdl_wait(); waited = true; }
                 uint32_t bytes = 0;
                 int page_of_tile[4];
 #pragma unroll
                 for (int j = 0; j < 4; ++j) {
                     page_of_tile[j] = -1;
                     if (j < n_tiles) {
-                        const int base = (kt0 + j) * 16;
+                        const int base = tiles.at(kt0 + j) * 16;
                         const int page = pt.page_of(p.page_shift >= 0 ? base >> p.page_shift : base / p.page_size);
                         if (page >= 0 && page < p.num_pages) { page_of_tile[j] = page; bytes += 2 * RING_TILE_BYTES; }
                     }
@@ -1316,7 +1320,7 @@ __global__ void __launch_bounds__(160, 2) fa_decode_ring_kernel(const __grid_con
 #pragma unroll
                 for (int j = 0; j < 4; ++j) {
                     if (page_of_tile[j] < 0) continue;
-                    const int base = (kt0 + j) * 16;
+                    const int base = tiles.at(kt0 + j) * 16;
                     const int slot = p.page_shift >= 0 ? base & (p.page_size - 1) : base % p.page_size;
                     const int row_k = ((page_of_tile[j] * 2) * p.num_kv_heads + geo.kvh) * p.page_size + slot;
                     const int row_v = row_k + p.num_kv_heads * p.page_size;
@@ -1359,7 +1363,7 @@ __global__ void __launch_bounds__(160, 2) fa_decode_ring_kernel(const __grid_con
             KeyTile tile;
             tile.base = -1;
             if (kt < tile_end) {
-                const int base = kt * 16;
+                const int base = tiles.at(kt) * 16;
                 const int page = pt.page_of(p.page_shift >= 0 ? base >> p.page_shift : base / p.page_size);
                 if (page >= 0 && page < p.num_pages) ring_take_keys(ring + s * RING_STAGE_BYTES + warp * 2 * RING_TILE_BYTES, base, last_pos, tile);
                 else if (lane == 0 && p.error_flag) atomicExch(p.error_flag, 3);
@@ -1432,13 +1436,13 @@ MLB_EXPORT int mlb_fa_max_splits() { return MAX_SPLITS; }
 MLB_EXPORT int mlb_paged_attention_mma(const void* q, const void* pages, void* out, const int* seq_starts,
                                        const int* seq_pos0, const int* block_table, const int* work, int num_work,
                                        int max_blocks, int num_pages, int page_size, int num_heads, int num_kv_heads,
-                                       int window, int chunk, float scale, int mode, int splits, const float* sink, float softcap,
+                                       int window, int keep, int chunk, float scale, int mode, int splits, const float* sink, float softcap,
                                        const float* distance_bias, int last_distance, int* error_flag, cudaStream_t stream) {
     if (num_heads <= 0 || num_kv_heads <= 0 || num_heads % num_kv_heads != 0)
         return fail(MLB_INVALID_ARGUMENT, "paged_attention_mma: bad head counts %d/%d", num_heads, num_kv_heads);
     if (page_size <= 0 || page_size % 16 != 0)
         return fail(MLB_UNSUPPORTED_SIZE, "paged_attention_mma: page_size %d must be a multiple of 16", page_size);
-    if (num_pages <= 0 || max_blocks <= 0 || window < 0 || chunk < 0 || num_work < 0)
+    if (num_pages <= 0 || max_blocks <= 0 || window < 0 || keep < 0 || chunk < 0 || num_work < 0)
         return fail(MLB_INVALID_ARGUMENT, "paged_attention_mma: bad cache geometry");
     const bool force_ring = (mode & 4) != 0, forbid_ring = (mode & 8) != 0;
     mode &= 3;
@@ -1451,7 +1455,7 @@ MLB_EXPORT int mlb_paged_attention_mma(const void* q, const void* pages, void* o
     if (num_work == 0) return MLB_OK;
     FaParams p{(const __nv_bfloat16*)q, (const __nv_bfloat16*)pages, (__nv_bfloat16*)out, seq_starts, seq_pos0,
                block_table, work, max_blocks, num_pages, page_size, num_heads, num_kv_heads,
-               num_heads / num_kv_heads, chunk, window, softcap > 0.0f ? softcap * LOG2E : scale * LOG2E,
+               num_heads / num_kv_heads, chunk, window, keep, softcap > 0.0f ? softcap * LOG2E : scale * LOG2E,
                (page_size & (page_size - 1)) == 0 ? __builtin_ctz((unsigned)page_size) : -1, error_flag,
                mode == 2 ? 1 : 0, softcap > 0.0f ? scale / softcap : 0.0f, sink, DistanceBias{distance_bias, last_distance}};
     if (distance_bias && last_distance < 0) return fail(MLB_INVALID_ARGUMENT, "paged_attention_mma: a distance bias has a last distance");

@@ -16,7 +16,7 @@
 //                S of tile j+1 is issued before P V of tile j, so the tensor pipe works on
 //                the next scores while the softmax warps turn the current ones into P.
 //     warps 2-5  softmax, one thread per query row: tcgen05.ld brings the row's 128 scores,
-//                mask (only in tiles that touch the causal or window edge), running maximum and
+//                mask (only in tiles that touch the causal edge, the window's or the kept first tokens'), running maximum and
 //                sum in fp32 with base-2 exponentials, P rounded to bf16 and written back to
 //                tensor memory (tcgen05.st, two buffers, two keys per column): it never touches
 //                shared memory.  The accumulator in tensor memory is rescaled
@@ -76,7 +76,7 @@ struct TcParams {
     const int* block_table;         // [A, max_blocks]
     const int* work;                // [num_work, 2] (sequence, 128-row tile of its new tokens)
     int max_blocks, num_pages, page_size, pages_per_tile;
-    int num_heads, num_kv_heads, group, window, chunk;
+    int num_heads, num_kv_heads, group, window, keep, chunk;   // keep: the first tokens that stay visible in front of the window
     float scale_log2;               // softmax scale * log2(e); with a cap on the scores: cap * log2(e)
     int* error_flag;
     float cap_pre;                  // > 0: scores are capped, s <- cap * tanh(s * scale / cap); this is scale / cap
@@ -249,8 +249,8 @@ fa_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_con
     const int rows = min(BM, n_new - row_first);
     const int qpos_first = pos0 + row_first, qpos_last = qpos_first + rows - 1;
     const int lo = first_visible_key(qpos_first, p.window, p.chunk);
-    const int kt_begin = lo / BN;
-    const int n_tiles = qpos_last / BN + 1 - kt_begin;
+    const KeyTiles tiles = key_tiles(lo, qpos_last, p.keep, BN);
+    const int n_tiles = tiles.count;
     const int kvh = head / p.group;
 
     // Ring items in order of need: K0, then for every tile j: K(j+1) if there is one, V(j).
@@ -274,7 +274,7 @@ fa_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_con
         };
         auto lookup = [&](int i) {                        // lane g: the page of block g of item i's tile
             int is_v;
-            const int block = (kt_begin + tile_of(i, is_v)) * p.pages_per_tile + lane;
+            const int block = tiles.at(tile_of(i, is_v)) * p.pages_per_tile + lane;
             return (lane < p.pages_per_tile && block < p.max_blocks) ? __ldg(table + block) : -1;
         };
         bool ok = true;
@@ -293,11 +293,11 @@ fa_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_con
             if (lane == 0) mbar_expect_tx(bar, KV_BYTES);
             __syncwarp();
             if (lane < p.pages_per_tile) {
-                const int block = (kt_begin + tile) * p.pages_per_tile + lane;
+                const int block = tiles.at(tile) * p.pages_per_tile + lane;
                 if (page < 0 || page >= p.num_pages) {
                     // a page that holds a key some row must see has to exist; the others are masked
                     const int first_key = block * p.page_size;
-                    if (first_key <= qpos_last && first_key + p.page_size - 1 >= lo && p.error_flag) atomicExch(p.error_flag, 2);
+                    if (first_key <= qpos_last && (first_key + p.page_size - 1 >= lo || first_key < p.keep) && p.error_flag) atomicExch(p.error_flag, 2);
                     page = 0;
                 }
                 const int row = ((page * 2 + is_v) * p.num_kv_heads + kvh) * p.page_size;
@@ -406,7 +406,7 @@ fa_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_con
                     sr[c] = __float_as_uint(fmaf(-2.0f, rcp, 1.0f));
                 }
             }
-            const int kbase = (kt_begin + j) * BN;
+            const int kbase = tiles.at(j) * BN;
             // a bias by distance: one number for a tile all of whose distances lie at or beyond the table's last one, else
             // it is added score by score (in base-2 units, so that scale and offset below are 1 and 0)
             float sc = p.scale_log2, off = 0.0f;
@@ -424,13 +424,13 @@ fa_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_con
                     sc = 1.0f;
                 }
             }
-            const bool edge = (kbase + BN - 1 > qpos_first) || (kbase < first_visible_key(qpos_last, p.window, p.chunk));
+            const bool edge = (kbase + BN - 1 > qpos_first) || (kbase < first_visible_key(qpos_last, p.window, p.chunk) && kbase + BN > p.keep);
             float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};       // four chains: no 128-long dependence
             if (edge) {
 #pragma unroll
                 for (int c = 0; c < BN; ++c) {
                     const int kpos = kbase + c;
-                    const float s = (kpos <= qpos && kpos >= lo_r) ? __uint_as_float(sr[c]) : -INFINITY;
+                    const float s = key_visible(kpos, qpos, lo_r, p.keep) ? __uint_as_float(sr[c]) : -INFINITY;
                     sr[c] = __float_as_uint(s);
                     mx4[c & 3] = fmaxf(mx4[c & 3], s);
                 }
@@ -476,18 +476,19 @@ fa_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_con
                 ok = wait_all(&pv_done[j & 1], ((j - 2) >> 1) & 1, 30);
                 if (!ok) break;
             }
-            // Keys outside lo..hi of the whole tile have P = 0, but 0 * V must not be NaN whatever an unused
+            // Keys that no row of the tile sees (behind the newest one; between the kept first ones and the window) have P = 0, but 0 * V must not be NaN whatever an unused
             // slot of a page holds: their V rows are cleared before the tensor core reads them.
-            const int keep_from = max(0, lo - kbase), keep_to = min(BN, qpos_last + 1 - kbase);
-            if (keep_from > 0 || keep_to < BN) {
+            const int gap_from = min(BN, max(0, p.keep - kbase)), gap = max(0, min(BN, lo - kbase) - gap_from);
+            const int keep_to = min(BN, qpos_last + 1 - kbase);
+            if (gap > 0 || keep_to < BN) {
                 const int v_item = (j + 1 < n_tiles) ? 2 * j + 2 : 2 * j + 1;
                 ok = wait_all(&slot_full[v_item % SLOTS], (v_item / SLOTS) & 1, 32);
                 if (!ok) break;
                 const uint32_t vb = ring_s + (v_item % SLOTS) * KV_BYTES;
-                const int cleared = keep_from + (BN - keep_to);
+                const int cleared = gap + (BN - keep_to);
                 for (int i = r; i < cleared * SPANS * 8; i += BM) {
                     const int row_i = i / (SPANS * 8), rest = i % (SPANS * 8);
-                    const int key = row_i < keep_from ? row_i : keep_to + (row_i - keep_from);
+                    const int key = row_i < gap ? gap_from + row_i : keep_to + (row_i - gap);
                     const uint32_t addr = vb + (rest / 8) * (BN * ROW_BYTES) + key * ROW_BYTES + (rest % 8) * 16;
                     asm volatile("st.shared.v4.b32 [%0], {%1, %1, %1, %1};" ::"r"(addr), "r"(0u) : "memory");
                 }
@@ -597,12 +598,12 @@ MLB_EXPORT int mlb_fa_tc_supported(int page_size, float scale) {
 MLB_EXPORT int mlb_paged_attention_tc(const void* q, long long ldq, const void* pages, void* out, long long ldo, int tokens,
                                       const int* seq_starts, const int* seq_pos0, const int* block_table, const int* work,
                                       int num_work, int max_blocks, int num_pages, int page_size, int num_heads,
-                                      int num_kv_heads, int window, int chunk, float scale, const float* sink, float softcap,
+                                      int num_kv_heads, int window, int keep, int chunk, float scale, const float* sink, float softcap,
                                       const float* distance_bias, int last_distance, int* error_flag, cudaStream_t stream) {
     if (num_heads <= 0 || num_kv_heads <= 0 || num_heads % num_kv_heads != 0)
         return fail(MLB_INVALID_ARGUMENT, "attention_tc: bad head counts %d/%d", num_heads, num_kv_heads);
     if (!mlb_fa_tc_supported(page_size, scale)) return MLB_UNSUPPORTED_SIZE;
-    if (num_pages <= 0 || max_blocks <= 0 || window < 0 || chunk < 0 || num_work < 0 || tokens < 0)
+    if (num_pages <= 0 || max_blocks <= 0 || window < 0 || keep < 0 || chunk < 0 || num_work < 0 || tokens < 0)
         return fail(MLB_INVALID_ARGUMENT, "attention_tc: bad cache geometry");
     if (ldq < (long long)num_heads * D || ldo < (long long)num_heads * D || ldq % 8 != 0 || ldo % 8 != 0 ||
         ((uintptr_t)q & 15) || ((uintptr_t)out & 15) || ((uintptr_t)pages & 15))
@@ -619,7 +620,7 @@ MLB_EXPORT int mlb_paged_attention_tc(const void* q, long long ldq, const void* 
     if (status != MLB_OK) return status;
 
     TcParams p{(__nv_bfloat16*)out, ldo, seq_starts, seq_pos0, block_table, work, max_blocks, num_pages, page_size,
-               BN / page_size, num_heads, num_kv_heads, num_heads / num_kv_heads, window, chunk,
+               BN / page_size, num_heads, num_kv_heads, num_heads / num_kv_heads, window, keep, chunk,
                softcap > 0.0f ? softcap * LOG2E : scale * LOG2E, error_flag, softcap > 0.0f ? scale / softcap : 0.0f, sink,
                DistanceBias{distance_bias, last_distance}};
     if (distance_bias && last_distance < 0) return fail(MLB_INVALID_ARGUMENT, "attention_tc: a distance bias has a last distance");

@@ -92,6 +92,24 @@ __device__ __forceinline__ int first_visible_key(int pos, int window, int chunk)
     return lo;
 }
 
+// Does a query at position `pos`, whose window starts at `lo`, see the key at `key`?  `keep`: the first tokens of a sequence
+// that stay visible in front of the window (0: none).
+__device__ __forceinline__ bool key_visible(int key, int pos, int lo, int keep) { return key <= pos && (key >= lo || key < keep); }
+
+// The key tiles (of `width` keys, at multiples of `width`) that hold a visible key: those of the kept first tokens, then
+// those from the window's start to the last key, numbered through without the gap between them.
+struct KeyTiles {
+    int kept, first, count;
+    __device__ __forceinline__ int at(int i) const { return i < kept ? i : first + (i - kept); }
+};
+__device__ __forceinline__ KeyTiles key_tiles(int lo, int last, int keep, int width) {
+    KeyTiles t;
+    t.first = lo / width;
+    t.kept = min((keep + width - 1) / width, t.first);
+    t.count = t.kept + last / width - t.first + 1;
+    return t;
+}
+
 // A score bias that depends on the distance query - key and on the head: one row a head, the values of distances 0, 1, ..
 // last with DISTANCE_PAD copies of the first value in front and DISTANCE_PAD copies of the last one behind (every distance
 // beyond `last` has the last one's value), so that a tile's distances around a row's end need no bounds of their own.

@@ -109,7 +109,8 @@ __global__ void __launch_bounds__(WARPS * 32) delta_prepare_kernel(PrepareParams
 
 // ------------------------------------------------------------------------------ the recurrence
 struct ScanParams {
-    const float* qn; const float* kn;        // [T, G * DK]
+    const float* qn; const float* kn;        // [T, G * DK], rows ld_qk apart
+    long long ld_qk;
     const float* g;                          // [T, H * DK]
     const float* beta;                       // [T, H]: beta of the delta rule, w of rule 3 (null: 1); else unused and may be null
     const float* bonus;                      // [H, DK] (rule 2 only)
@@ -188,12 +189,12 @@ __global__ void __launch_bounds__(COLS * LANES) delta_scan_kernel(ScanParams p) 
         for (int i = 0; i < ROWS; ++i) U[i] = row_of(i) < p.DK ? p.bonus[(size_t)h * p.DK + row_of(i)] : 0.0f;
     }
 
-    const float* const q_base = p.qn + ((size_t)start * p.G + kvh) * p.DK;
-    const float* const k_base = p.kn + ((size_t)start * p.G + kvh) * p.DK;
+    const float* const q_base = p.qn + (size_t)start * p.ld_qk + (size_t)kvh * p.DK;
+    const float* const k_base = p.kn + (size_t)start * p.ld_qk + (size_t)kvh * p.DK;
     const float* const g_base = RULE == RULE_HEAD_DECAY ? p.g + (size_t)start * p.g_pitch + h : p.g + ((size_t)start * p.H + h) * p.DK;
     const float* const v_base = p.v + (size_t)start * p.ld_v + (size_t)h * p.DV;
     const float* const b_base = p.beta ? p.beta + (size_t)start * p.H + h : g_base;     // without beta: any readable address, the value is unused
-    const size_t qk_pitch = (size_t)p.G * p.DK, g_pitch = (size_t)p.H * p.DK;
+    const size_t qk_pitch = (size_t)p.ld_qk, g_pitch = (size_t)p.H * p.DK;
     // the chunk that begins at token `first` into staging buffer `buf`; padding (rows beyond DK, columns beyond DV) becomes
     // zero: a zero k and q keep such rows of S at zero whatever g is.  Tokens beyond the sequence's are not staged (nor read).
     auto stage = [&](int first, int buf) {
@@ -458,7 +459,7 @@ template <int RULE>
 int launch_scan(const float* qn, const float* kn, const float* g, const float* beta, const float* bonus, const float* v, long long ld_v,
                 float* o, float* state, const int* slots, int num_slots, const int* seq_starts, const int* seq_pos0,
                 int A, int H, int G, int DK, int DV, int* error_flag, cudaStream_t stream, int g_pitch = 0, float* n_state = nullptr,
-                float* den = nullptr) {
+                float* den = nullptr, long long ld_qk = 0) {
     if (A < 0 || H <= 0 || G <= 0 || H % G || DK <= 0 || DK > MAX_D || DV <= 0)
         return fail(MLB_UNSUPPORTED_SIZE, "scan: heads %d/%d, widths %d (at most %d) / %d", H, G, DK, MAX_D, DV);
     if (!qn || !kn || !g || (RULE == RULE_DELTA && !beta) || (RULE == RULE_BONUS_READ && !bonus) || !v || !o || !state || !slots ||
@@ -466,8 +467,10 @@ int launch_scan(const float* qn, const float* kn, const float* g, const float* b
         return fail(MLB_INVALID_ARGUMENT, "scan: null operand");
     if (A == 0) return MLB_OK;
     const bool aligned = ((uintptr_t)qn | (uintptr_t)kn | (RULE == RULE_HEAD_DECAY ? 0 : (uintptr_t)g) | (uintptr_t)v) % 16 == 0;
-    const int vec = aligned && DK % 4 == 0 && DV % 4 == 0 && ld_v % 4 == 0;
-    ScanParams p{qn, kn, g, beta, bonus, v, ld_v, o, state, slots, num_slots, seq_starts, seq_pos0, A, H, G, DK, DV,
+    if (ld_qk == 0) ld_qk = (long long)G * DK;
+    if (ld_qk < (long long)G * DK) return fail(MLB_INVALID_ARGUMENT, "scan: q and k rows overlap");
+    const int vec = aligned && DK % 4 == 0 && DV % 4 == 0 && ld_v % 4 == 0 && ld_qk % 4 == 0;
+    ScanParams p{qn, kn, ld_qk, g, beta, bonus, v, ld_v, o, state, slots, num_slots, seq_starts, seq_pos0, A, H, G, DK, DV,
                  g_pitch, n_state, den, vec, error_flag};
     // A handful of long-running CTAs (a prompt portion: one CTA walks all its tokens) must be spread one to an SM.  Started
     // early behind a predecessor that still fills the SMs, they land wherever a slot falls free, several on one SM, and
@@ -512,13 +515,13 @@ MLB_EXPORT int mlb_linear_scan(int rule, const float* q, const float* k, const f
 }
 
 // rule 3: S <- g S + w k v^T, o = S^T q.  g [T, H] (per_token 1) or [H] (0, fixed); w [T, H] or null (1).  n_state [slots, H, DK] and
-// den [T, H] together: n <- g n + w k, den = n . q.
-MLB_EXPORT int mlb_head_scan(const float* q, const float* k, const float* g, int per_token, const float* w, const float* v, long long ld_v,
+// den [T, H] together: n <- g n + w k, den = n . q.  q, k [T, G * DK] with rows ld_qk apart; head h reads q/k head h / (H / G).
+MLB_EXPORT int mlb_head_scan(const float* q, const float* k, long long ld_qk, int G, const float* g, int per_token, const float* w, const float* v, long long ld_v,
                              float* o, float* state, float* n_state, float* den, const int* slots, int num_slots, const int* seq_starts,
                              const int* seq_pos0, int A, int H, int DK, int DV, int* error_flag, cudaStream_t stream) {
     if ((n_state == nullptr) != (den == nullptr)) return fail(MLB_INVALID_ARGUMENT, "head_scan: the vector's state and its read-out come together");
-    return launch_scan<RULE_HEAD_DECAY>(q, k, g, w, nullptr, v, ld_v, o, state, slots, num_slots, seq_starts, seq_pos0, A, H, H, DK, DV, error_flag,
-                                        stream, per_token ? H : 0, n_state, den);
+    return launch_scan<RULE_HEAD_DECAY>(q, k, g, w, nullptr, v, ld_v, o, state, slots, num_slots, seq_starts, seq_pos0, A, H, G, DK, DV, error_flag,
+                                        stream, per_token ? H : 0, n_state, den, ld_qk);
 }
 
 MLB_EXPORT int mlb_delta_output(const float* o, const float* weight, const float* proj, long long ld_proj, int n_partials,

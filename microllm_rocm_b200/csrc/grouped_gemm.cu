@@ -11,7 +11,8 @@
 // Each output element is accumulated by ONE thread over k = 0..K-1 in increasing order with fp32 FMA, so its value
 // depends neither on the tile it falls in nor on which other rows its group holds: the fp32 path stays
 // bit-stable, and the bf16 path (bf16 operands, fp32 accumulation) differs from it only by the operands' rounding.
-// The optional epilogue multiplies by a factor read from an fp32 matrix at the output's own (row, column).
+// The optional epilogue multiplies by a factor read from an fp32 matrix at the output's own (row, column), or by a number
+// per entry of the row list.
 #include "common.cuh"
 
 using namespace mlb;
@@ -32,6 +33,7 @@ struct GroupedParams {
     const int* c_rows;
     int a_row_div;
     const float* factor; long long ldf;      // null: no epilogue
+    const float* row_scale;                  // [entries of a_rows], null: 1
     int M, N, K, G;
 };
 
@@ -44,6 +46,7 @@ grouped_gemm_kernel(GroupedParams p) {
     __shared__ float Ws[BK][BN + 4];
     __shared__ int src_row[BM];
     __shared__ int dst_row[BM];
+    __shared__ float row_scale_s[BM];
     __shared__ int tile_info[3];             // group, first place, places in this tile
     __shared__ int offsets_s[MAX_GROUPS + 1];
     const int tid = threadIdx.x;
@@ -81,6 +84,7 @@ grouped_gemm_kernel(GroupedParams p) {
             c = p.c_rows ? p.c_rows[place] : place;
         }
         src_row[tid] = a; dst_row[tid] = c;
+        row_scale_s[tid] = (p.row_scale && tid < count) ? p.row_scale[p.a_rows ? p.a_rows[first + tid] : first + tid] : 1.0f;
     }
     __syncthreads();
     const AT* A = (const AT*)p.A + (size_t)group * p.a_group_cols;
@@ -135,6 +139,7 @@ grouped_gemm_kernel(GroupedParams p) {
             if (n >= p.N) continue;
             const size_t col = (size_t)group * p.c_group_cols + n;
             float v = acc[i][j];
+            if (p.row_scale) v *= row_scale_s[ty * TM + i];
             if (p.factor) v *= p.factor[(size_t)c * p.ldf + col];
             ((OutT*)p.C)[(size_t)c * p.ldc + col] = from_f32<OutT>(v);
         }
@@ -154,14 +159,14 @@ void launch(const GroupedParams& p, int row_tile, unsigned tiles_y, cudaStream_t
 MLB_EXPORT int mlb_grouped_gemm(const void* A, long long lda, long long a_group_cols, const void* W, long long ldw,
                                 long long w_group_stride, void* C, long long ldc, long long c_group_cols,
                                 const int* group_offsets, const int* a_rows, const int* c_rows, int a_row_div,
-                                const float* factor, long long ldf, int M, int N, int K, int G, int dtype, int out_dtype,
+                                const float* factor, long long ldf, const float* row_scale, int M, int N, int K, int G, int dtype, int out_dtype,
                                 int row_tile, cudaStream_t stream) {
     if (M < 0 || N <= 0 || K <= 0 || G <= 0 || a_row_div <= 0 || (row_tile != 16 && row_tile != 64))
         return fail(MLB_INVALID_ARGUMENT, "grouped_gemm: bad sizes M=%d N=%d K=%d G=%d", M, N, K, G);
     if (group_offsets && G > MAX_GROUPS) return fail(MLB_UNSUPPORTED_SIZE, "grouped_gemm: more than %d groups", MAX_GROUPS);
     if (M == 0) return MLB_OK;
     GroupedParams p{A, lda, a_group_cols, W, ldw, w_group_stride, C, ldc, c_group_cols, group_offsets, a_rows, c_rows,
-                    a_row_div, factor, ldf, M, N, K, G};
+                    a_row_div, factor, ldf, row_scale, M, N, K, G};
     const long long per = (M + row_tile - 1) / row_tile;
     const long long tiles = group_offsets ? per + G : per * G;
     if (tiles > 65535) return fail(MLB_UNSUPPORTED_SIZE, "grouped_gemm: %lld row tiles exceed one launch", tiles);

@@ -9,7 +9,8 @@
 // bytes, which keeps the eight rows of an ldmatrix phase in different banks.
 // Epilogues: none; times a factor read at the output's own place (fp32); or DUAL: the weight holds two row blocks
 // (gate rows, then `dual_rows` further down the up rows), both are multiplied in the same pass and the result is
-// silu(gate) * up (or the clamped form, gated_value).
+// silu(gate) * up (or the clamped form, gated_value), optionally with both products times a number per entry of the row list
+// first (a weight on the row that goes in, applied in fp32 behind the product).
 // Sizes must suit 16-byte pieces (K, the row pitches and the column blocks multiples of 8 elements); the caller
 // sends everything else to the CUDA-core kernel.
 #include "common.cuh"
@@ -35,6 +36,7 @@ struct MmaParams {
     long long dual_rows;                       // DUAL: the second row block starts this many rows further down
     int M, N, K, G;
     int act;                                   // DUAL: the activation (gated_value)
+    const float* row_scale;                    // DUAL: both products times row_scale[a_rows[place]] (null: 1)
 };
 
 __device__ __forceinline__ void cp_async16(void* dst, const void* src, bool valid) {
@@ -67,7 +69,7 @@ __device__ __forceinline__ float gated_value(float g, float u, int act) {
 
 __host__ __device__ constexpr int threads_of(int bm) { return bm == 128 ? 256 : 128; }
 constexpr size_t smem_of(int bm, bool dual) {
-    return (size_t)STAGES * (bm + (dual ? 2 : 1) * BN) * (bk_of(bm, dual) + 8) * sizeof(__nv_bfloat16) + (2 * bm + 4 + MAX_GROUPS + 1) * sizeof(int);
+    return (size_t)STAGES * (bm + (dual ? 2 : 1) * BN) * (bk_of(bm, dual) + 8) * sizeof(__nv_bfloat16) + (3 * bm + 4 + MAX_GROUPS + 1) * sizeof(int);
 }
 
 template <typename OutT, int BM, bool DUAL>
@@ -89,7 +91,8 @@ grouped_mma_kernel(MmaParams p) {
     WTile Ws = reinterpret_cast<WTile>(smem_raw + (size_t)STAGES * BM * PITCH * sizeof(__nv_bfloat16));   // [STAGES][NB][BN][PITCH]
     int* src_row = reinterpret_cast<int*>(smem_raw + (size_t)STAGES * (BM + NB * BN) * PITCH * sizeof(__nv_bfloat16));
     int* dst_row = src_row + BM;
-    int* tile_info = dst_row + BM;
+    float* row_scale_s = reinterpret_cast<float*>(dst_row + BM);
+    int* tile_info = dst_row + 2 * BM;
     int* offsets_s = tile_info + 4;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     if (p.group_offsets) {                           // fetched by all threads at once, walked by one
@@ -126,6 +129,7 @@ grouped_mma_kernel(MmaParams p) {
             c = p.c_rows ? p.c_rows[place] : place;
         }
         src_row[tid] = a; dst_row[tid] = c;
+        if (DUAL) row_scale_s[tid] = (p.row_scale && tid < count) ? p.row_scale[p.a_rows ? p.a_rows[first + tid] : first + tid] : 1.0f;
     }
     __syncthreads();
     const __nv_bfloat16* A = p.A + (size_t)group * p.a_group_cols;
@@ -229,8 +233,10 @@ grouped_mma_kernel(MmaParams p) {
     for (int m = 0; m < MT; ++m)
 #pragma unroll
     for (int half = 0; half < 2; ++half) {
-        const int c = dst_row[warp_m * 16 * MT + 16 * m + (lane >> 2) + 8 * half];
+        const int row = warp_m * 16 * MT + 16 * m + (lane >> 2) + 8 * half;
+        const int c = dst_row[row];
         if (c < 0) continue;
+        const float by = DUAL ? row_scale_s[row] : 1.0f;
 #pragma unroll
         for (int j = 0; j < NT; ++j)
 #pragma unroll
@@ -239,7 +245,7 @@ grouped_mma_kernel(MmaParams p) {
                 if (n >= p.N) continue;
                 const size_t col = (size_t)group * p.c_group_cols + n;
                 float v = acc[m][0][j][half * 2 + i];
-                if (DUAL) v = gated_value(v, acc[m][NB - 1][j][half * 2 + i], p.act);
+                if (DUAL) v = gated_value(v * by, acc[m][NB - 1][j][half * 2 + i] * by, p.act);
                 if (p.factor) v *= p.factor[(size_t)c * p.ldf + col];
                 ((OutT*)p.C)[(size_t)c * p.ldc + col] = from_f32<OutT>(v);
             }
@@ -273,16 +279,17 @@ MLB_EXPORT int mlb_grouped_mma(const void* A, long long lda, long long a_group_c
                                long long w_group_stride, void* C, long long ldc, long long c_group_cols,
                                const int* group_offsets, const int* a_rows, const int* c_rows, int a_row_div,
                                const float* factor, long long ldf, long long dual_rows, int M, int N, int K, int G,
-                               int out_dtype, int row_tile, int act, cudaStream_t stream) {
+                               int out_dtype, int row_tile, int act, const float* row_scale, cudaStream_t stream) {
     if (M < 0 || N <= 0 || K <= 0 || G <= 0 || a_row_div <= 0 || dual_rows < 0 || (row_tile != 16 && row_tile != 64 && row_tile != 128))
         return fail(MLB_INVALID_ARGUMENT, "grouped_mma: bad sizes M=%d N=%d K=%d G=%d", M, N, K, G);
     if (K % 8 || lda % 8 || ldw % 8 || a_group_cols % 8 || w_group_stride % 8 || (uintptr_t)A % 16 || (uintptr_t)W % 16)
         return fail(MLB_UNSUPPORTED_SIZE, "grouped_mma: K, the row pitches and the column blocks must be multiples of 8 elements");
     if (act < 0 || act == 1) return fail(MLB_INVALID_ARGUMENT, "grouped_mma: unknown activation %d", act);
+    if (row_scale && dual_rows == 0) return fail(MLB_INVALID_ARGUMENT, "grouped_mma: a factor per row goes with the two-block product");
     if (group_offsets && G > MAX_GROUPS) return fail(MLB_UNSUPPORTED_SIZE, "grouped_mma: more than %d groups", MAX_GROUPS);
     if (M == 0) return MLB_OK;
     MmaParams p{(const __nv_bfloat16*)A, lda, a_group_cols, (const __nv_bfloat16*)W, ldw, w_group_stride, C, ldc, c_group_cols,
-                group_offsets, a_rows, c_rows, a_row_div, factor, ldf, dual_rows, M, N, K, G, act};
+                group_offsets, a_rows, c_rows, a_row_div, factor, ldf, dual_rows, M, N, K, G, act, row_scale};
     const long long per = (M + row_tile - 1) / row_tile;
     const long long tiles = group_offsets ? per + G : per * G;
     if (tiles > 65535) return fail(MLB_UNSUPPORTED_SIZE, "grouped_mma: %lld row tiles exceed one launch", tiles);

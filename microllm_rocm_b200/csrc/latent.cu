@@ -18,7 +18,10 @@
 //                       q_full[T, H*(R+Dr)]         only its last Dr columns per head: the rotated query parts
 //                       pages[page, slot, 0:R]      c = rms(latent) * norm_weight;  [R:R+Dr] = rotated kr
 //                       gate_out[T, gate_width]     sigmoid of the pre-activations, fp32
-//                    rotation: element i of the first rot_dims is paired with i + rot_dims/2, angle = pos * inv_freq[i]
+//                    rotation: element i of the first rot_dims is paired with i + rot_dims/2 (or, interleaved, 2i with 2i + 1),
+//                    angle = pos * inv_freq[pair], cosines and sines times `magnitude`
+//   latent_compress  for queries that come out of a latent of their own (a product follows before latent_prepare can split
+//                    them): the cache row as above, and c_q[T, RQ] = rms(columns cq_col..) * its weight in the compute dtype
 //   latent_attention_plain   one warp per (token, head); keys in tiles of 32 at absolute multiples of 32, running
 //                    maximum and sum in fp32; a learned per-head sink enters the denominator once, unscaled, with
 //                    no value.  Bit-stable under any cutting of the tokens into steps.
@@ -35,11 +38,25 @@ struct PrepareParams {
     long long q_col, kv_col, gate_col;
     const float* norm_weight; float eps;
     const int* positions; const int* token_seq; const int* block_table; int max_blocks;
-    const float* inv_freq; int rot_dims;
+    const float* inv_freq; int rot_dims; int interleaved; float magnitude;
     void* q_plain; void* q_full; void* pages; float* gate_out;
     int num_pages, page_size, tokens, heads, dim, rot_dim, rank, gate_width;
     int* error_flag;
+    // latent_compress only
+    long long cq_col; int cq_rank; const float* cq_weight; void* cq_out;
 };
+
+// where the partner of element i of a rotated part sits, which pair they are, and whether i is the pair's first element
+struct Pair { int other, index; bool first; };
+__device__ __forceinline__ Pair pair_of(int i, int half, int interleaved) {
+    if (interleaved) return Pair{i ^ 1, i >> 1, (i & 1) == 0};
+    return i < half ? Pair{i + half, i, true} : Pair{i - half, i - half, false};
+}
+
+__device__ __forceinline__ float turned(float v, float other, bool first, float angle, float magnitude) {
+    const float cs = cosf(angle) * magnitude, sn = sinf(angle) * magnitude;
+    return first ? v * cs - other * sn : v * cs + other * sn;
+}
 
 __device__ __forceinline__ float proj_at(const PrepareParams& p, size_t row_base, long long col) {
     float v = p.proj[row_base + col];
@@ -48,6 +65,47 @@ __device__ __forceinline__ float proj_at(const PrepareParams& p, size_t row_base
 }
 
 constexpr int SLICE = 1024;        // query and gate columns per block
+
+// The token's cache row: the normalised latent, then the shared key part with its rotation.
+template <typename KVT>
+__device__ __forceinline__ void store_cache_row(const PrepareParams& p, int t, size_t row, int pos, float* scratch) {
+    const int half = p.rot_dims / 2;
+    const int Dk = p.rank + p.rot_dim;
+    KVT* cache_row = nullptr;
+    if (p.pages) {
+        const int block = pos / p.page_size;
+        const int page = block < p.max_blocks ? p.block_table[(size_t)p.token_seq[t] * p.max_blocks + block] : -1;
+        if (page < 0 || page >= p.num_pages) {
+            if (threadIdx.x == 0 && p.error_flag) atomicExch(p.error_flag, 1);
+        } else {
+            cache_row = (KVT*)p.pages + ((size_t)page * p.page_size + pos % p.page_size) * Dk;
+        }
+        // the latent, divided by its root mean square, times the norm's weight
+        float ss = 0.0f;
+        for (int c = threadIdx.x; c < p.rank; c += blockDim.x) {
+            const float v = proj_at(p, row, p.kv_col + c);
+            ss += v * v;
+        }
+        ss = block_sum(ss, scratch);
+        const float inv = 1.0f / sqrtf(ss / (float)p.rank + p.eps);
+        if (cache_row) {
+            for (int c = threadIdx.x; c < p.rank; c += blockDim.x)
+                cache_row[c] = from_f32<KVT>(proj_at(p, row, p.kv_col + c) * inv * p.norm_weight[c]);
+            // the shared key part: its first rot_dims elements turned in pairs, the rest passed on
+            for (int i = threadIdx.x; i < p.rot_dim; i += blockDim.x) {
+                float out;
+                const float v = proj_at(p, row, p.kv_col + p.rank + i);
+                if (i < p.rot_dims) {
+                    const Pair pr = pair_of(i, half, p.interleaved);
+                    out = turned(v, proj_at(p, row, p.kv_col + p.rank + pr.other), pr.first, (float)pos * p.inv_freq[pr.index], p.magnitude);
+                } else {
+                    out = v;
+                }
+                cache_row[p.rank + i] = from_f32<KVT>(out);
+            }
+        }
+    }
+}
 
 template <typename QT, typename KVT>
 __global__ void __launch_bounds__(256)
@@ -82,54 +140,37 @@ latent_prepare_kernel(PrepareParams p) {
             const int r = i - p.dim;
             float out = v;
             if (r < p.rot_dims) {
-                const int pair = r < half ? r : r - half;
-                const float angle = (float)pos * p.inv_freq[pair];
-                const float cs = cosf(angle), sn = sinf(angle);
-                const float other = proj_at(p, row, p.q_col + (long long)h * per_head + p.dim + (r < half ? r + half : r - half));
-                out = r < half ? v * cs - other * sn : v * cs + other * sn;
+                const Pair pr = pair_of(r, half, p.interleaved);
+                const float other = proj_at(p, row, p.q_col + (long long)h * per_head + p.dim + pr.other);
+                out = turned(v, other, pr.first, (float)pos * p.inv_freq[pr.index], p.magnitude);
             }
             ((QT*)p.q_full)[((size_t)t * p.heads + h) * Dk + p.rank + r] = from_f32<QT>(out);
         }
         return;
     }
-    // where this token's cache row lives
-    KVT* cache_row = nullptr;
-    if (p.pages) {
-        const int block = pos / p.page_size;
-        const int page = block < p.max_blocks ? p.block_table[(size_t)p.token_seq[t] * p.max_blocks + block] : -1;
-        if (page < 0 || page >= p.num_pages) {
-            if (threadIdx.x == 0 && p.error_flag) atomicExch(p.error_flag, 1);
-        } else {
-            cache_row = (KVT*)p.pages + ((size_t)page * p.page_size + pos % p.page_size) * Dk;
-        }
-        // the latent, divided by its root mean square, times the norm's weight
-        float ss = 0.0f;
-        for (int c = threadIdx.x; c < p.rank; c += blockDim.x) {
-            const float v = proj_at(p, row, p.kv_col + c);
-            ss += v * v;
-        }
-        ss = block_sum(ss, scratch);
-        const float inv = 1.0f / sqrtf(ss / (float)p.rank + p.eps);
-        if (cache_row) {
-            for (int c = threadIdx.x; c < p.rank; c += blockDim.x)
-                cache_row[c] = from_f32<KVT>(proj_at(p, row, p.kv_col + c) * inv * p.norm_weight[c]);
-            // the shared key part: pairs (i, i + half) of its first rot_dims turned, the rest passed on
-            for (int i = threadIdx.x; i < p.rot_dim; i += blockDim.x) {
-                float out;
-                const float v = proj_at(p, row, p.kv_col + p.rank + i);
-                if (i < p.rot_dims) {
-                    const int pair = i < half ? i : i - half;
-                    const float angle = (float)pos * p.inv_freq[pair];
-                    const float cs = cosf(angle), sn = sinf(angle);
-                    const float other = proj_at(p, row, p.kv_col + p.rank + (i < half ? i + half : i - half));
-                    out = i < half ? v * cs - other * sn : v * cs + other * sn;
-                } else {
-                    out = v;
-                }
-                cache_row[p.rank + i] = from_f32<KVT>(out);
-            }
-        }
+    store_cache_row<KVT>(p, t, row, pos, scratch);
+}
+
+// One block per token and part: blockIdx.y 0 the cache row, 1 the queries' latent.
+template <typename QT, typename KVT>
+__global__ void __launch_bounds__(256)
+latent_compress_kernel(PrepareParams p) {
+    pdl_prologue();
+    __shared__ float scratch[32];
+    const int t = blockIdx.x;
+    const size_t row = (size_t)t * p.ld;
+    if (blockIdx.y == 0) {
+        store_cache_row<KVT>(p, t, row, p.positions[t], scratch);
+        return;
     }
+    float ss = 0.0f;
+    for (int c = threadIdx.x; c < p.cq_rank; c += blockDim.x) {
+        const float v = proj_at(p, row, p.cq_col + c);
+        ss = fmaf(v, v, ss);
+    }
+    const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)p.cq_rank + p.eps);
+    for (int c = threadIdx.x; c < p.cq_rank; c += blockDim.x)
+        ((QT*)p.cq_out)[(size_t)t * p.cq_rank + c] = from_f32<QT>(proj_at(p, row, p.cq_col + c) * inv * p.cq_weight[c]);
 }
 
 constexpr int WARPS = 4;
@@ -229,7 +270,7 @@ latent_attention_plain_kernel(AttnParams p) {
 MLB_EXPORT int mlb_latent_prepare(const float* proj, long long ld, int n_partials, long long partial_stride, long long q_col,
                                   long long kv_col, long long gate_col, const float* norm_weight, float eps,
                                   const int* positions, const int* token_seq, const int* block_table, int max_blocks,
-                                  const float* inv_freq, int rot_dims, void* q_plain, void* q_full, int q_dtype, void* pages,
+                                  const float* inv_freq, int rot_dims, int interleaved, float magnitude, void* q_plain, void* q_full, int q_dtype, void* pages,
                                   int kv_dtype, float* gate_out, int num_pages, int page_size, int tokens, int heads, int dim,
                                   int rot_dim, int rank, int gate_width, int* error_flag, cudaStream_t stream) {
     if (tokens < 0 || heads <= 0 || dim <= 0 || rot_dim < 0 || rank <= 0 || n_partials < 1 || !(eps > 0.0f))
@@ -238,8 +279,8 @@ MLB_EXPORT int mlb_latent_prepare(const float* proj, long long ld, int n_partial
     if (pages && (page_size <= 0 || num_pages <= 0 || max_blocks <= 0)) return fail(MLB_INVALID_ARGUMENT, "latent_prepare: bad cache geometry");
     if (tokens == 0) return MLB_OK;
     PrepareParams p{proj, ld, n_partials, partial_stride, q_col, kv_col, gate_col, norm_weight, eps, positions, token_seq,
-                    block_table, max_blocks, inv_freq, rot_dims, q_plain, q_full, pages, gate_out, num_pages, page_size,
-                    tokens, heads, dim, rot_dim, rank, gate_width, error_flag};
+                    block_table, max_blocks, inv_freq, rot_dims, interleaved, magnitude, q_plain, q_full, pages, gate_out, num_pages, page_size,
+                    tokens, heads, dim, rot_dim, rank, gate_width, error_flag, 0, 0, nullptr, nullptr};
     const int columns = heads * (dim + rot_dim) + (gate_out ? gate_width : 0);
     const dim3 grid(tokens, 1 + (columns + SLICE - 1) / SLICE);
     if (q_dtype == MLB_F32 && (kv_dtype == MLB_F32 || !pages))
@@ -249,6 +290,31 @@ MLB_EXPORT int mlb_latent_prepare(const float* proj, long long ld, int n_partial
     else
         return fail(MLB_INVALID_ARGUMENT, "latent_prepare: unsupported dtypes %d / %d", q_dtype, kv_dtype);
     return check_launch("latent_prepare");
+}
+
+// the cache row of every token (pages may be null: none is stored) and c_q [tokens, cq_rank] out of one projection
+MLB_EXPORT int mlb_latent_compress(const float* proj, long long ld, int n_partials, long long partial_stride, long long cq_col, int cq_rank,
+                                   const float* cq_weight, void* cq_out, int q_dtype, long long kv_col, const float* norm_weight, float eps,
+                                   const int* positions, const int* token_seq, const int* block_table, int max_blocks,
+                                   const float* inv_freq, int rot_dims, int interleaved, float magnitude, void* pages, int kv_dtype,
+                                   int num_pages, int page_size, int tokens, int rot_dim, int rank, int* error_flag, cudaStream_t stream) {
+    if (tokens < 0 || cq_rank <= 0 || rot_dim < 0 || rank <= 0 || n_partials < 1 || !(eps > 0.0f) || !proj || !cq_weight || !cq_out || !norm_weight)
+        return fail(MLB_INVALID_ARGUMENT, "latent_compress: bad operands");
+    if (rot_dims < 0 || rot_dims % 2 || rot_dims > rot_dim) return fail(MLB_INVALID_ARGUMENT, "latent_compress: rot_dims %d must be even and at most %d", rot_dims, rot_dim);
+    if (pages && (page_size <= 0 || num_pages <= 0 || max_blocks <= 0)) return fail(MLB_INVALID_ARGUMENT, "latent_compress: bad cache geometry");
+    if (tokens == 0) return MLB_OK;
+    PrepareParams p{};
+    p.proj = proj; p.ld = ld; p.n_partials = n_partials; p.partial_stride = partial_stride; p.kv_col = kv_col; p.norm_weight = norm_weight; p.eps = eps;
+    p.positions = positions; p.token_seq = token_seq; p.block_table = block_table; p.max_blocks = max_blocks; p.inv_freq = inv_freq;
+    p.rot_dims = rot_dims; p.interleaved = interleaved; p.magnitude = magnitude; p.pages = pages; p.num_pages = num_pages; p.page_size = page_size;
+    p.tokens = tokens; p.rot_dim = rot_dim; p.rank = rank; p.error_flag = error_flag;
+    p.cq_col = cq_col; p.cq_rank = cq_rank; p.cq_weight = cq_weight; p.cq_out = cq_out;
+    const dim3 grid(tokens, 2);
+    if (q_dtype == MLB_F32 && (kv_dtype == MLB_F32 || !pages)) launch_kernel(latent_compress_kernel<float, float>, grid, 256, 0, stream, p);
+    else if (q_dtype == MLB_BF16 && (kv_dtype == MLB_BF16 || !pages))
+        launch_kernel(latent_compress_kernel<__nv_bfloat16, __nv_bfloat16>, grid, 256, 0, stream, p);
+    else return fail(MLB_INVALID_ARGUMENT, "latent_compress: unsupported dtypes %d / %d", q_dtype, kv_dtype);
+    return check_launch("latent_compress");
 }
 
 MLB_EXPORT int mlb_latent_attention_plain(const void* q, int q_dtype, const void* pages, int kv_dtype, void* out, int out_dtype,

@@ -8,13 +8,15 @@
 //                 `scoring` 2: s = sigmoid(z); the experts form `groups` equal groups of neighbours, a group scores the sum of its
 //                 two largest s[e] + b[e] and only experts of the `keep` best groups can be chosen; the `top` largest of those
 //                 run with weights s / (sum of the chosen s + 1e-20) * weight_scale.
+//                 `scoring` 3: the same with the chosen s * weight_scale as the weights, not divided by their sum.
 //   moe_align     (below) skips, without raising the flag, ids in [experts, experts + passthrough): outputs of the router that
 //                 have no expert behind them (moe_combine adds the token's own input times the weight for those).
 //   moe_align     from ids[T*top] to a list of the pairs (token, choice) sorted by expert: offsets[E+1] and
 //                 sorted[T*top] (pair indices); the order inside an expert is arbitrary, every pair's result is
-//                 computed on its own.
+//                 computed on its own.  Optionally dest[T*top]: place i's row in a [top, T] layout, (pair % top) * T + pair / top,
+//                 for results that are to be added up as `top` partial results of all tokens.
 //   moe_combine   out[t,:] = (sum_j w[t,j] * y[t*top + j,:] + g[t] * sum_k shared_k[t,:]) * s[:]
-//                 j in order of choice; shared (may be split partial sums), g and s are optional.
+//                 j in order of choice; shared (may be split partial sums), g and s are optional; without weights w = 1.
 #include "common.cuh"
 
 using namespace mlb;
@@ -39,15 +41,15 @@ moe_select_kernel(const float* __restrict__ logits, long long ld, int n_partials
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int t = blockIdx.x * ROUTE_WARPS + warp;
     if (t >= tokens) return;
-    float* z = logits_s + (size_t)warp * experts * (scoring + 1);
-    float* score = z + experts;                         // scoring 1 and 2 only
+    float* z = logits_s + (size_t)warp * experts * (min(scoring, 2) + 1);
+    float* score = z + experts;                         // scoring 1 to 3 only
     const float* row = logits + (size_t)t * ld;
     for (int e = lane; e < experts; e += 32) {
         float v = row[e];
         for (int k = 1; k < n_partials; ++k) v += row[(size_t)k * partial_stride + e];
         z[e] = scoring >= 1 ? v : v + (bias ? bias[e] : 0.0f);
     }
-    if (scoring == 2) {
+    if (scoring >= 2) {
         for (int e = lane; e < experts; e += 32) {      // (every lane turns its own elements)
             const float v = z[e], sc = v >= 0.0f ? 1.0f / (1.0f + expf(-v)) : expf(v) / (1.0f + expf(v));
             score[e] = sc;
@@ -123,6 +125,10 @@ moe_select_kernel(const float* __restrict__ logits, long long ld, int n_partials
         if (lane < top) weights[(size_t)t * top + lane] = chosen;
         return;
     }
+    if (scoring == 3) {
+        if (lane < top) weights[(size_t)t * top + lane] = chosen * weight_scale;
+        return;
+    }
     if (scoring == 2) {
         const float total = warp_sum(lane < top ? chosen : 0.0f) + 1e-20f;
         if (lane < top) weights[(size_t)t * top + lane] = chosen / total * weight_scale;
@@ -135,7 +141,7 @@ moe_select_kernel(const float* __restrict__ logits, long long ld, int n_partials
 
 __global__ void __launch_bounds__(1024)
 moe_align_kernel(const int* __restrict__ ids, int pairs, int experts, int* __restrict__ offsets, int* __restrict__ sorted,
-                 int* __restrict__ error_flag, int passthrough) {
+                 int* __restrict__ error_flag, int passthrough, int* __restrict__ dest, int top) {
     pdl_prologue();
     __shared__ int count[MAX_EXPERTS];
     __shared__ int cursor[MAX_EXPERTS];
@@ -155,7 +161,11 @@ moe_align_kernel(const int* __restrict__ ids, int pairs, int experts, int* __res
     __syncthreads();
     for (int i = threadIdx.x; i < pairs; i += blockDim.x) {
         const int e = ids[i];
-        if (e >= 0 && e < experts) sorted[atomicAdd(&cursor[e], 1)] = i;
+        if (e >= 0 && e < experts) {
+            const int place = atomicAdd(&cursor[e], 1);
+            sorted[place] = i;
+            if (dest) dest[place] = (i % top) * (pairs / top) + i / top;
+        }
     }
 }
 
@@ -173,10 +183,10 @@ __global__ void moe_combine_kernel(const float* __restrict__ y, const float* __r
         const float own = x_dtype == MLB_BF16 ? to_f32(((const __nv_bfloat16*)x)[i]) : ((const float*)x)[i];
         for (int j = 0; j < top; ++j) {
             const float v = ids[(size_t)t * top + j] >= experts ? own : y[((size_t)t * top + j) * width + c];
-            acc = fmaf(weights[(size_t)t * top + j], v, acc);
+            acc = fmaf(weights ? weights[(size_t)t * top + j] : 1.0f, v, acc);
         }
     } else
-    for (int j = 0; j < top; ++j) acc = fmaf(weights[(size_t)t * top + j], y[((size_t)t * top + j) * width + c], acc);
+    for (int j = 0; j < top; ++j) acc = fmaf(weights ? weights[(size_t)t * top + j] : 1.0f, y[((size_t)t * top + j) * width + c], acc);
     if (shared) {
         float s = shared[i];
         for (int k = 1; k < n_shared; ++k) s += shared[(size_t)k * shared_stride + i];
@@ -190,24 +200,24 @@ __global__ void moe_combine_kernel(const float* __restrict__ y, const float* __r
 MLB_EXPORT int mlb_moe_select(const float* logits, long long ld, int n_partials, long long partial_stride, const float* bias,
                               int gate_col, int tokens, int experts, int top, int* ids, float* weights, float* gate_out,
                               int scoring, int groups, int keep, float weight_scale, cudaStream_t stream) {
-    if (scoring < 0 || scoring > 2) return fail(MLB_INVALID_ARGUMENT, "moe_select: unknown scoring %d", scoring);
-    if (scoring == 2 && (groups <= 0 || experts % groups || keep <= 0 || keep > groups || top > keep * (experts / groups)))
+    if (scoring < 0 || scoring > 3) return fail(MLB_INVALID_ARGUMENT, "moe_select: unknown scoring %d", scoring);
+    if (scoring >= 2 && (groups <= 0 || experts % groups || keep <= 0 || keep > groups || top > keep * (experts / groups)))
         return fail(MLB_INVALID_ARGUMENT, "moe_select: %d of %d groups of %d experts, top %d", keep, groups, experts, top);
     if (tokens < 0 || experts <= 0 || experts > MAX_EXPERTS || top <= 0 || top > experts || top > MAX_TOP || n_partials < 1 ||
         ld < experts || gate_col >= ld)
         return fail(MLB_INVALID_ARGUMENT, "moe_select: bad sizes (experts %d, top %d; at most %d and %d)", experts, top, MAX_EXPERTS, MAX_TOP);
     if (tokens == 0) return MLB_OK;
     const unsigned blocks = (tokens + ROUTE_WARPS - 1) / ROUTE_WARPS;
-    launch_kernel(moe_select_kernel, blocks, ROUTE_WARPS * 32, (size_t)ROUTE_WARPS * experts * sizeof(float) * (scoring + 1),
+    launch_kernel(moe_select_kernel, blocks, ROUTE_WARPS * 32, (size_t)ROUTE_WARPS * experts * sizeof(float) * ((scoring < 2 ? scoring : 2) + 1),
                   stream, logits, ld, n_partials, partial_stride, bias, gate_col, tokens, experts, top, ids, weights, gate_out, scoring, groups, keep,
                   weight_scale);
     return check_launch("moe_select");
 }
 
 MLB_EXPORT int mlb_moe_align(const int* ids, int pairs, int experts, int* offsets, int* sorted, int* error_flag, int passthrough,
-                             cudaStream_t stream) {
-    if (pairs < 0 || experts <= 0 || experts > MAX_EXPERTS || passthrough < 0) return fail(MLB_INVALID_ARGUMENT, "moe_align: bad sizes");
-    launch_kernel(moe_align_kernel, 1, 1024, 0, stream, ids, pairs, experts, offsets, sorted, error_flag, passthrough);
+                             int* dest, int top, cudaStream_t stream) {
+    if (pairs < 0 || experts <= 0 || experts > MAX_EXPERTS || passthrough < 0 || (dest && (top <= 0 || pairs % top))) return fail(MLB_INVALID_ARGUMENT, "moe_align: bad sizes");
+    launch_kernel(moe_align_kernel, 1, 1024, 0, stream, ids, pairs, experts, offsets, sorted, error_flag, passthrough, dest, top);
     return check_launch("moe_align");
 }
 

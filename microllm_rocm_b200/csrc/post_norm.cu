@@ -3,7 +3,8 @@
 //   mlb_normed_add_rmsnorm   d = s1 * sum_k d1[k][r] + s2 * sum_k d2[k][r]        (d2 optional: two mixers side by side)
 //                            x[r] += d / sqrt(mean(d^2) + eps) * w_post            in place, the residual stream
 //                            out[r] = x[r] / sqrt(mean(x[r]^2) + eps) * w_next     optional: the norm in front of the next
-//                                                                                  sublayer, stored in the compute dtype
+//                                                                                  sublayer, stored in the compute dtype;
+//                            without w_next out[r] = x[r] in the compute dtype (sublayers that read the stream itself)
 //
 // d1/d2 may be K-split partial results, added in split order.  One block of a fixed size per row, reductions in a fixed tree: a
 // row's result depends on the row alone.  Rows of up to 4,096 columns stay in registers (up to sixteen columns a thread,
@@ -24,7 +25,7 @@ struct PostNormParams {
     const float* d1; int n1; long long stride1; float s1;
     const float* d2; int n2; long long stride2; float s2;
     const float* w_post; const float* w_next;
-    void* out;                // compute dtype, may be null (then w_next is unused)
+    void* out;                // compute dtype, may be null (then w_next is unused); w_next null: the stream itself
     int width; float eps;
 };
 
@@ -58,8 +59,12 @@ __global__ void __launch_bounds__(PN_THREADS) normed_add_rmsnorm_kernel(PostNorm
         ss2 = fmaf(x, x, ss2);
     }
     if (!p.out) return;
-    const float inv2 = 1.0f / sqrtf(block_sum(ss2, scratch) / (float)W + p.eps);
     OutT* yr = (OutT*)p.out + r * W;
+    if (!p.w_next) {
+        for (int c = threadIdx.x; c < W; c += PN_THREADS) yr[c] = from_f32<OutT>(row_s[c]);      // (what this thread wrote itself)
+        return;
+    }
+    const float inv2 = 1.0f / sqrtf(block_sum(ss2, scratch) / (float)W + p.eps);
     for (int c = threadIdx.x; c < W; c += PN_THREADS) yr[c] = from_f32<OutT>(row_s[c] * inv2 * p.w_next[c]);
 }
 
@@ -75,7 +80,7 @@ __global__ void __launch_bounds__(PN_THREADS) normed_add_rmsnorm_reg_kernel(Post
     for (int i = 0; i < PER; ++i) {            // weights: no kernel of a step writes them
         const int c = threadIdx.x + i * PN_THREADS;
         wp[i] = c < W ? p.w_post[c] : 0.0f;
-        wn[i] = (p.out && c < W) ? p.w_next[c] : 0.0f;
+        wn[i] = (p.out && p.w_next && c < W) ? p.w_next[c] : 0.0f;
     }
     pdl_wait();
     float* xr = p.x + r * W;
@@ -120,8 +125,16 @@ __global__ void __launch_bounds__(PN_THREADS) normed_add_rmsnorm_reg_kernel(Post
         ss2 = fmaf(x[i], x[i], ss2);
     }
     if (!p.out) return;
-    const float inv2 = 1.0f / sqrtf(block_sum(ss2, scratch) / (float)W + p.eps);
     OutT* yr = (OutT*)p.out + r * W;
+    if (!p.w_next) {
+#pragma unroll
+        for (int i = 0; i < PER; ++i) {
+            const int c = threadIdx.x + i * PN_THREADS;
+            if (c < W) yr[c] = from_f32<OutT>(x[i]);
+        }
+        return;
+    }
+    const float inv2 = 1.0f / sqrtf(block_sum(ss2, scratch) / (float)W + p.eps);
 #pragma unroll
     for (int i = 0; i < PER; ++i) {
         const int c = threadIdx.x + i * PN_THREADS;
@@ -145,7 +158,7 @@ int launch_in_registers(const PostNormParams& p, int rows, cudaStream_t stream) 
 MLB_EXPORT int mlb_normed_add_rmsnorm(float* x, const float* d1, int n1, long long stride1, float s1, const float* d2, int n2,
                                       long long stride2, float s2, const float* w_post, const float* w_next, void* out,
                                       int out_dtype, int rows, int width, float eps, cudaStream_t stream) {
-    if (rows < 0 || width <= 0 || !x || !d1 || n1 < 1 || (d2 && n2 < 1) || !w_post || (out && !w_next))
+    if (rows < 0 || width <= 0 || !x || !d1 || n1 < 1 || (d2 && n2 < 1) || !w_post)
         return fail(MLB_INVALID_ARGUMENT, "normed_add_rmsnorm: bad operands");
     const size_t smem = (size_t)width * sizeof(float);
     if (smem > 200 * 1024) return fail(MLB_UNSUPPORTED_SIZE, "normed_add_rmsnorm: width %d", width);

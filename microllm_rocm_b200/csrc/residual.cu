@@ -8,7 +8,7 @@
 //
 //   bigram_add            x[t,:] += table[row(t),:], row = (previous token * a + token * b) mod n, or row n for a sequence's
 //                         first token; the previous token of a step's first token is the sequence's state (one int per slot).
-//                         Given the token table as well, x[t,:] = tokens[id[t],:] + table[row(t),:] in one pass (bad id -> NaN).
+//                         Given the token table as well, x[t,:] = tokens[id[t],:] * scale + table[row(t),:] in one pass (bad id -> NaN).
 //   bigram_state          state[slot of a] = the last token sequence a brought in this step
 //   softcap_rows          x <- cap * tanh(x / cap) in place
 //
@@ -164,7 +164,7 @@ MLB_EXPORT int mlb_stream_entry(float* x, const float* x0, const float* v, int w
 namespace {
 
 template <typename TableT>
-__global__ void bigram_add_kernel(float* __restrict__ x, const TableT* __restrict__ table, const TableT* __restrict__ token_table, int vocab,
+__global__ void bigram_add_kernel(float* __restrict__ x, const TableT* __restrict__ table, const TableT* __restrict__ token_table, int vocab, float scale,
                                   const int* __restrict__ ids,
                                   const int* __restrict__ token_seq, const int* __restrict__ seq_starts, const int* __restrict__ seq_pos0,
                                   const int* __restrict__ state, const int* __restrict__ slots, int num_slots, int tokens, int width,
@@ -193,7 +193,7 @@ __global__ void bigram_add_kernel(float* __restrict__ x, const TableT* __restric
             return;
         }
         const TableT* own = token_table + (size_t)id * width;
-        for (int c = threadIdx.x; c < width; c += blockDim.x) dst[c] = to_f32(own[c]) + to_f32(src[c]);
+        for (int c = threadIdx.x; c < width; c += blockDim.x) dst[c] = fmaf(to_f32(own[c]), scale, to_f32(src[c]));
         return;
     }
     for (int c = threadIdx.x; c < width; c += blockDim.x) dst[c] += to_f32(src[c]);
@@ -216,7 +216,7 @@ __global__ void softcap_rows_kernel(float* __restrict__ x, long long n, float ca
 
 }  // namespace
 
-MLB_EXPORT int mlb_bigram_add(float* x, const void* table, int table_dtype, const void* token_table, int vocab, const int* ids, const int* token_seq, const int* seq_starts,
+MLB_EXPORT int mlb_bigram_add(float* x, const void* table, int table_dtype, const void* token_table, int vocab, float scale, const int* ids, const int* token_seq, const int* seq_starts,
                               const int* seq_pos0, int* state, const int* slots, int num_slots, int tokens, int num_seqs, int width,
                               int buckets, int mul_prev, int mul_cur, int update_state, int* error_flag, cudaStream_t stream) {
     if (tokens < 0 || num_seqs < 0 || width <= 0 || buckets <= 0 || num_slots <= 0 || !x || !table || !ids || !state || !slots)
@@ -225,10 +225,10 @@ MLB_EXPORT int mlb_bigram_add(float* x, const void* table, int table_dtype, cons
     const int threads = width >= 1024 ? 256 : 128;
     if (table_dtype == MLB_BF16)
         launch_kernel(bigram_add_kernel<__nv_bfloat16>, (unsigned)tokens, threads, 0, stream, x, (const __nv_bfloat16*)table,
-                      (const __nv_bfloat16*)token_table, vocab, ids, token_seq,
+                      (const __nv_bfloat16*)token_table, vocab, scale, ids, token_seq,
                       seq_starts, seq_pos0, (const int*)state, slots, num_slots, tokens, width, buckets, (long long)mul_prev, (long long)mul_cur, error_flag);
     else if (table_dtype == MLB_F32)
-        launch_kernel(bigram_add_kernel<float>, (unsigned)tokens, threads, 0, stream, x, (const float*)table, (const float*)token_table, vocab,
+        launch_kernel(bigram_add_kernel<float>, (unsigned)tokens, threads, 0, stream, x, (const float*)table, (const float*)token_table, vocab, scale,
                       ids, token_seq, seq_starts,
                       seq_pos0, (const int*)state, slots, num_slots, tokens, width, buckets, (long long)mul_prev, (long long)mul_cur, error_flag);
     else return fail(MLB_INVALID_ARGUMENT, "bigram_add: unsupported table dtype %d", table_dtype);

@@ -1,6 +1,7 @@
 // Short causal convolution over time, per channel, with the last taps - 1 inputs of every sequence kept as state:
 //
-//   y[t, c] = act( sum_j w[c, j] * u[t - taps + 1 + j, c] ),   u = 0 before the sequence's start, act = identity | silu
+//   y[t, c] = act( bias[c] + sum_j w[c, j] * u[t - taps + 1 + j, c] ),  (bias optional)
+//         u = 0 before the sequence's start, act = identity | silu
 //
 // u is a block of columns of a projection's fp32 output (or of its K-split partial results, added in split
 // order).  Tokens of a step are the flat batch of the engine: a sequence's tokens are consecutive, it held `pos0`
@@ -31,6 +32,7 @@ struct ConvParams {
     int T, A, C, taps, act;
     int* error_flag;
     int run = 1;               // tokens a thread of the four-channel kernel walks
+    const float* bias = nullptr;   // [C] or null
 };
 
 __device__ __forceinline__ float input_at(const ConvParams& p, long long row, int c) {
@@ -60,6 +62,7 @@ __global__ void short_conv_kernel(ConvParams p) {
         else if (pos0 + src >= 0 && slot_ok) u = p.state[((size_t)slot * hist + (hist + src)) * p.C + c];
         acc = fmaf(p.w[(size_t)c * p.taps + j], u, acc);
     }
+    if (p.bias) acc += p.bias[c];
     if (p.act == 1) acc = acc / (1.0f + expf(-acc));
     p.y[(size_t)t * p.ldy + c] = acc;
 }
@@ -92,6 +95,7 @@ __global__ void short_conv_x4_kernel(ConvParams p) {
     float wreg[4 * TAPS];               // the weights are never written by a kernel: fetched before the wait for the predecessor
 #pragma unroll
     for (int k = 0; k < 4 * TAPS; ++k) wreg[k] = p.w[(size_t)c * TAPS + k];
+    const float4 shift = p.bias ? *reinterpret_cast<const float4*>(p.bias + c) : make_float4(0.f, 0.f, 0.f, 0.f);
     pdl_wait();
     if (!active) return;
     const int t0 = (int)(i / C4) * p.run;
@@ -125,6 +129,7 @@ __global__ void short_conv_x4_kernel(ConvParams p) {
                 acc.z = fmaf(wreg[2 * TAPS + j], u.z, acc.z); acc.w = fmaf(wreg[3 * TAPS + j], u.w, acc.w);
             }
         }
+        acc.x += shift.x; acc.y += shift.y; acc.z += shift.z; acc.w += shift.w;
         if (p.act == 1) {
             acc.x = acc.x / (1.0f + expf(-acc.x)); acc.y = acc.y / (1.0f + expf(-acc.y));
             acc.z = acc.z / (1.0f + expf(-acc.z)); acc.w = acc.w / (1.0f + expf(-acc.w));
@@ -171,17 +176,18 @@ int check(const ConvParams& p, const char* what) {
 }  // namespace
 
 MLB_EXPORT int mlb_short_conv(const float* u, long long ld, int n_partials, long long partial_stride, int col0, const float* w,
-                              float* state, const int* slots, int num_slots, const int* seq_starts, const int* seq_pos0,
+                              const float* bias, float* state, const int* slots, int num_slots, const int* seq_starts, const int* seq_pos0,
                               const int* token_seq, float* y, long long ldy, int T, int A, int C, int taps, int act,
                               int* error_flag, cudaStream_t stream) {
     ConvParams p{u, ld, n_partials, partial_stride, col0, w, state, slots, num_slots, seq_starts, seq_pos0, token_seq, y, ldy,
                  T, A, C, taps, act, error_flag};
     if (int s = check(p, "short_conv")) return s;
+    p.bias = bias;
     if (!y) return fail(MLB_INVALID_ARGUMENT, "short_conv: null output");
     if (T == 0) return MLB_OK;
     const long long n = (long long)T * C;
     const bool x4 = C % 4 == 0 && ld % 4 == 0 && ldy % 4 == 0 && col0 % 4 == 0 && partial_stride % 4 == 0 &&
-                    ((uintptr_t)u | (uintptr_t)y | (uintptr_t)state) % 16 == 0;
+                    ((uintptr_t)u | (uintptr_t)y | (uintptr_t)state | (uintptr_t)bias) % 16 == 0;
     p.run = T >= 64 * CONV_RUN ? CONV_RUN : 1;
     const long long x4_threads = ((long long)T + p.run - 1) / p.run * (C / 4);
     const unsigned x4_blocks = (unsigned)((x4_threads + 127) / 128);

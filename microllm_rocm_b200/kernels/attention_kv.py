@@ -26,7 +26,7 @@ ops.register_signatures("attention_kv.cu", {
     "mlb_row_norm_columns": [c_void_p, c_longlong, c_int, c_longlong, c_int, c_int, c_int, c_int, c_void_p, c_int, c_int, c_void_p, c_float,
                              c_void_p, c_void_p],
     "mlb_paged_attention_kv": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
-                               c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_longlong, c_int, c_longlong, c_int,
+                               c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_longlong, c_int, c_longlong, c_int,
                                c_int, c_void_p, c_float, c_void_p, c_int, c_void_p, c_void_p],
 })
 
@@ -140,8 +140,8 @@ def paged_attention_kv(q: torch.Tensor, pages: torch.Tensor, out: torch.Tensor, 
                        block_table: torch.Tensor, page_size: int, heads: int, kv_heads: int, dk: int, dv: int, scale: float,
                        window: Optional[int], gate: Optional[torch.Tensor], gate_col: int,
                        error_flag: Optional[torch.Tensor], chunk: Optional[int] = None, gate_per_head: bool = False,
-                       sink: Optional[torch.Tensor] = None, softcap: float = 0.0, bias=None) -> None:
-    """`bias`: an `ops.DistanceBias`, added to the scaled score by head and distance.
+                       sink: Optional[torch.Tensor] = None, softcap: float = 0.0, bias=None, keep_first: int = 0) -> None:
+    """`keep_first`: the first tokens of a sequence that stay visible in front of the window.  `bias`: an `ops.DistanceBias`, added to the scaled score by head and distance.
     `chunk`: a query sees only the keys of its own block of `chunk` positions (blocks counted from position 0).
     `gate_per_head`: the gate has one column per head.  `sink` [heads] fp32: exp(sink) joins each head's denominator.
     `softcap` > 0: scores become softcap * tanh(score / softcap).
@@ -164,5 +164,5 @@ def paged_attention_kv(q: torch.Tensor, pages: torch.Tensor, out: torch.Tensor, 
     build.check(L, L.mlb_paged_attention_kv(
         q.data_ptr(), ops.dtype_tag(q), pages.data_ptr(), ops.dtype_tag(pages), out.data_ptr(), ops.dtype_tag(out),
         positions.data_ptr(), token_seq.data_ptr(), block_table.data_ptr(), block_table.shape[1], pages.shape[0], page_size, T,
-        heads, kv_heads, dk, dv, int(window or 0), int(chunk or 0), float(scale), g_ptr, g_ld, g_n, g_stride, int(gate_col),
+        heads, kv_heads, dk, dv, int(window or 0), int(keep_first), int(chunk or 0), float(scale), g_ptr, g_ld, g_n, g_stride, int(gate_col),
         1 if gate_per_head else 0, ops._ptr(sink), float(softcap or 0.0), *ops.distance_bias_args(bias, heads), ops._ptr(error_flag), ops._stream()))

@@ -17,7 +17,7 @@ from .build import KernelError
 SOURCE = "grouped_gemm.cu"
 ops.register_signatures(SOURCE, {
     "mlb_grouped_gemm": [c_void_p, c_longlong, c_longlong, c_void_p, c_longlong, c_longlong, c_void_p, c_longlong, c_longlong,
-                         c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_int, c_int,
+                         c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
                          c_int, c_void_p],
 })
 
@@ -26,7 +26,7 @@ MMA_SOURCE = "grouped_mma.cu"
 ops.register_signatures(MMA_SOURCE, {
     "mlb_grouped_mma": [c_void_p, c_longlong, c_longlong, c_void_p, c_longlong, c_longlong, c_void_p, c_longlong, c_longlong,
                         c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_longlong, c_longlong, c_int, c_int, c_int, c_int, c_int,
-                        c_int, c_int, c_void_p],
+                        c_int, c_int, c_void_p, c_void_p],
 })
 
 # Tests set it to False to send bf16 products to the CUDA-core kernel and compare.
@@ -57,14 +57,15 @@ def row_tile_for(rows: int, groups: int, listed: bool, tensor_cores: bool) -> in
 def grouped_linear(a: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, *, rows: int, a_group_cols: int = 0,
                    c_group_cols: int = 0, group_offsets: Optional[torch.Tensor] = None, a_rows: Optional[torch.Tensor] = None,
                    c_rows: Optional[torch.Tensor] = None, a_row_div: int = 1, factor: Optional[torch.Tensor] = None,
-                   row_tile: int = 64) -> None:
+                   row_scale: Optional[torch.Tensor] = None, row_tile: int = 64) -> None:
     """weight [G, N, K]; a [*, lda] and out [*, ldc] are 2-D and row-major.
 
     group g multiplies the K columns of `a` that start at g * a_group_cols with weight[g] and writes N columns of
     `out` starting at g * c_group_cols.  With `group_offsets` ([G + 1] int32 on the device) group g owns the places
     offsets[g]..offsets[g+1]-1 of a sorted list of `rows` places; `a_rows[place] // a_row_div` is the row read and
     `c_rows[place]` the row written (None: the place itself).  Without it every group takes rows 0..rows-1.
-    `factor` (fp32, the shape of `out`): the result is multiplied by it element by element."""
+    `factor` (fp32, the shape of `out`): the result is multiplied by it element by element.  `row_scale` (fp32, one number per
+    entry that a_rows may name): a row's result is multiplied by row_scale[a_rows[place]] (not on the tensor cores)."""
     ops._need(a, "a", dims=2); ops._need(weight, "weight", dims=3); ops._need(out, "out", dims=2)
     if a.dtype != weight.dtype:
         raise KernelError(f"grouped_linear: operands are {a.dtype} and {weight.dtype}")
@@ -80,29 +81,34 @@ def grouped_linear(a: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, *, 
         ops._need(factor, "factor", torch.float32, 2)
         if factor.shape[1] < out.shape[1]:
             raise KernelError("grouped_linear: the factor matrix is narrower than the output")
-    if row_tile == 128 and not mma_supported(a, weight, a_group_cols):
+    if row_scale is not None:
+        ops._need(row_scale, "row_scale", torch.float32)
+    tensor_cores = mma_supported(a, weight, a_group_cols) and row_scale is None
+    if row_tile == 128 and not tensor_cores:
         row_tile = 64
-    if mma_supported(a, weight, a_group_cols):
+    if tensor_cores:
         L = ops.lib(MMA_SOURCE)
         build.check(L, L.mlb_grouped_mma(
             a.data_ptr(), a.stride(0), a_group_cols, weight.data_ptr(), weight.stride(1), weight.stride(0), out.data_ptr(),
             out.stride(0), c_group_cols, ops._ptr(group_offsets), ops._ptr(a_rows), ops._ptr(c_rows), int(a_row_div),
             ops._ptr(factor), factor.stride(0) if factor is not None else 0, 0, int(rows), N, K, G, ops.dtype_tag(out),
-            int(row_tile), 0, ops._stream()))
+            int(row_tile), 0, None, ops._stream()))
         return
     L = ops.lib(SOURCE)
     build.check(L, L.mlb_grouped_gemm(
         a.data_ptr(), a.stride(0), a_group_cols, weight.data_ptr(), weight.stride(1), weight.stride(0), out.data_ptr(),
         out.stride(0), c_group_cols, ops._ptr(group_offsets), ops._ptr(a_rows), ops._ptr(c_rows), int(a_row_div),
-        ops._ptr(factor), factor.stride(0) if factor is not None else 0, int(rows), N, K, G, ops.dtype_tag(a),
+        ops._ptr(factor), factor.stride(0) if factor is not None else 0, ops._ptr(row_scale), int(rows), N, K, G, ops.dtype_tag(a),
         ops.dtype_tag(out), int(row_tile), ops._stream()))
 
 
 def grouped_silu_mul(a: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, *, rows: int, group_offsets: torch.Tensor,
                      a_rows: Optional[torch.Tensor] = None, a_row_div: int = 1, row_tile: int = 64, alloc=None,
-                     activation: str = "silu", limit: Optional[float] = None) -> None:
+                     activation: str = "silu", limit: Optional[float] = None, row_scale: Optional[torch.Tensor] = None) -> None:
     """weight [G, 2 * F, K]: per group F gate rows over F up rows; out[place] = silu(a gate^T) * (a up^T), [rows, F]; or,
-    with `activation` "clamped_swish" and its `limit`, the clamped form (ops.activation_code).
+    with `activation` "clamped_swish" and its `limit`, the clamped form (ops.activation_code).  `row_scale` (fp32, one number per
+    entry that a_rows may name): both products are multiplied by row_scale[a_rows[place]] in front of the activation, which is a
+    weight on the row that goes in.
     On the tensor cores both products and the activation are one kernel; otherwise the fused product leaves
     [rows, 2 * F] (from `alloc(shape, dtype)`) and the activation kernel follows."""
     ops._need(a, "a", dims=2); ops._need(weight, "weight", dims=3); ops._need(out, "out", dims=2)
@@ -112,6 +118,8 @@ def grouped_silu_mul(a: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, *
         raise KernelError(f"grouped_silu_mul: activation {activation!r}")
     if two_f % 2 or tuple(out.shape) != (rows, F):
         raise KernelError("grouped_silu_mul: the weight holds gate rows over up rows, the output one column per pair")
+    if row_scale is not None:
+        ops._need(row_scale, "row_scale", torch.float32)
     if mma_supported(a, weight):
         ops._need(group_offsets, "group_offsets", torch.int32, 1)
         if a_rows is not None:
@@ -120,9 +128,10 @@ def grouped_silu_mul(a: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, *
         build.check(L, L.mlb_grouped_mma(
             a.data_ptr(), a.stride(0), 0, weight.data_ptr(), weight.stride(1), weight.stride(0), out.data_ptr(), out.stride(0), 0,
             group_offsets.data_ptr(), ops._ptr(a_rows), None, int(a_row_div), None, 0, F, int(rows), F, K, G,
-            ops.dtype_tag(out), int(row_tile), ops.activation_code(activation, limit), ops._stream()))
+            ops.dtype_tag(out), int(row_tile), ops.activation_code(activation, limit), ops._ptr(row_scale), ops._stream()))
         return
     row_tile = min(row_tile, 64)
     gate_up = alloc((rows, two_f), a.dtype) if alloc is not None else torch.empty((rows, two_f), dtype=a.dtype, device=a.device)
-    grouped_linear(a, weight, gate_up, rows=rows, group_offsets=group_offsets, a_rows=a_rows, a_row_div=a_row_div, row_tile=row_tile)
+    grouped_linear(a, weight, gate_up, rows=rows, group_offsets=group_offsets, a_rows=a_rows, a_row_div=a_row_div, row_tile=row_tile,
+                   row_scale=row_scale)
     ops.gated_act_mul(gate_up, out, activation, limit)

@@ -13,8 +13,11 @@ from .build import KernelError
 SOURCE = "latent.cu"
 ops.register_signatures(SOURCE, {
     "mlb_latent_prepare": [c_void_p, c_longlong, c_int, c_longlong, c_longlong, c_longlong, c_longlong, c_void_p, c_float,
-                           c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int,
+                           c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_float, c_void_p, c_void_p, c_int, c_void_p, c_int,
                            c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
+    "mlb_latent_compress": [c_void_p, c_longlong, c_int, c_longlong, c_longlong, c_int, c_void_p, c_void_p, c_int, c_longlong, c_void_p,
+                            c_float, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_float, c_void_p, c_int, c_int, c_int,
+                            c_int, c_int, c_int, c_void_p, c_void_p],
     "mlb_latent_attention_plain": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
                                    c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p],
 })
@@ -126,7 +129,7 @@ def prepare(proj: torch.Tensor, *, q_col: int, kv_col: int, gate_col: int, norm_
             positions: torch.Tensor, token_seq: torch.Tensor, block_table: Optional[torch.Tensor], inv_freq: torch.Tensor,
             rot_dims: int, q_plain: torch.Tensor, q_full: torch.Tensor, pages: Optional[torch.Tensor],
             gate_out: Optional[torch.Tensor], heads: int, dim: int, rot_dim: int, rank: int,
-            error_flag: Optional[torch.Tensor]) -> None:
+            error_flag: Optional[torch.Tensor], interleaved: bool = False, magnitude: float = 1.0) -> None:
     """proj: the fused projection [T, N] fp32 or its [S, T, N] partial sums; see csrc/latent.cu for what goes where.
     pages [num_pages, page_size, rank + rot_dim]; None: a run that reads another run's cache stores nothing."""
     n_partials, stride = 1, 0
@@ -149,7 +152,7 @@ def prepare(proj: torch.Tensor, *, q_col: int, kv_col: int, gate_col: int, norm_
         gate_width = gate_out.shape[1]
         if gate_out.shape[0] != T:
             raise KernelError("latent.prepare: one gate row per token")
-    if max(q_col + heads * (dim + rot_dim), kv_col + rank + rot_dim, gate_col + gate_width) > first.shape[1]:
+    if max(q_col + heads * (dim + rot_dim), kv_col + rank + rot_dim if pages is not None else 0, gate_col + gate_width) > first.shape[1]:
         raise KernelError("latent.prepare: a column range runs past the projection")
     num_pages = page_size = max_blocks = 0
     if pages is not None:
@@ -162,9 +165,42 @@ def prepare(proj: torch.Tensor, *, q_col: int, kv_col: int, gate_col: int, norm_
     build.check(L, L.mlb_latent_prepare(
         first.data_ptr(), first.stride(0), n_partials, stride, q_col, kv_col, gate_col, norm_weight.data_ptr(), float(eps),
         positions.data_ptr(), token_seq.data_ptr(), ops._ptr(block_table), max_blocks, inv_freq.data_ptr(), int(rot_dims),
-        q_plain.data_ptr(), q_full.data_ptr(), ops.dtype_tag(q_plain), ops._ptr(pages),
+        1 if interleaved else 0, float(magnitude), q_plain.data_ptr(), q_full.data_ptr(), ops.dtype_tag(q_plain), ops._ptr(pages),
         ops.dtype_tag(pages) if pages is not None else ops.F32, ops._ptr(gate_out), num_pages, page_size, T, heads, dim,
         rot_dim, rank, gate_width, ops._ptr(error_flag), ops._stream()))
+
+
+def compress(proj: torch.Tensor, *, cq_col: int, cq_weight: torch.Tensor, cq_out: torch.Tensor, kv_col: int, norm_weight: torch.Tensor,
+             eps: float, positions: torch.Tensor, token_seq: torch.Tensor, block_table: Optional[torch.Tensor], inv_freq: torch.Tensor,
+             rot_dims: int, interleaved: bool, magnitude: float, pages: Optional[torch.Tensor], rot_dim: int, rank: int,
+             error_flag: Optional[torch.Tensor]) -> None:
+    """Out of one projection (fp32 rows or their partial sums): the token's cache row, as in `prepare`, and the queries' own latent
+    cq_out [T, RQ] = columns cq_col.. / rms * cq_weight in cq_out's dtype.  pages None: a run that stores nothing."""
+    n_partials, stride, first = 1, 0, proj
+    if proj.dim() == 3:
+        ops._need(proj, "proj", torch.float32, 3)
+        n_partials, stride, first = proj.shape[0], proj.shape[1] * proj.shape[2], proj[0]
+    ops._need(first, "proj", torch.float32, 2); ops._need(cq_out, "cq_out", dims=2)
+    ops._need(cq_weight, "cq_weight", torch.float32, 1); ops._need(norm_weight, "norm_weight", torch.float32, 1)
+    ops._need(inv_freq, "inv_freq", torch.float32, 1); ops._need(positions, "positions", torch.int32, 1)
+    T, width = first.shape
+    rq = cq_out.shape[1]
+    if (cq_out.shape[0] != T or cq_weight.shape[0] != rq or norm_weight.shape[0] != rank or inv_freq.shape[0] * 2 != rot_dims
+            or positions.shape[0] != T or max(cq_col + rq, kv_col + rank + rot_dim) > width):
+        raise KernelError("latent.compress: shapes do not agree")
+    num_pages = page_size = max_blocks = 0
+    if pages is not None:
+        ops._need(pages, "pages", dims=3); ops._need(block_table, "block_table", torch.int32, 2)
+        num_pages, page_size, page_width = pages.shape
+        if page_width != rank + rot_dim:
+            raise KernelError(f"latent.compress: pages {tuple(pages.shape)} do not hold rows of {rank} + {rot_dim}")
+        max_blocks = block_table.shape[1]
+    L = ops.lib(SOURCE)
+    build.check(L, L.mlb_latent_compress(
+        first.data_ptr(), first.stride(0), n_partials, stride, cq_col, rq, cq_weight.data_ptr(), cq_out.data_ptr(), ops.dtype_tag(cq_out),
+        kv_col, norm_weight.data_ptr(), float(eps), positions.data_ptr(), token_seq.data_ptr(), ops._ptr(block_table), max_blocks,
+        inv_freq.data_ptr(), int(rot_dims), 1 if interleaved else 0, float(magnitude), ops._ptr(pages),
+        ops.dtype_tag(pages) if pages is not None else ops.F32, num_pages, page_size, T, rot_dim, rank, ops._ptr(error_flag), ops._stream()))
 
 
 def attention_plain(q: torch.Tensor, pages: torch.Tensor, out: torch.Tensor, sink: Optional[torch.Tensor],

@@ -91,7 +91,7 @@ _SIGNATURES = {
                                    c_float, c_void_p],
         "mlb_add_scaled_inplace": [c_void_p, c_void_p, c_int, c_longlong, c_void_p, c_int, c_longlong, c_void_p],
         "mlb_stream_entry": [c_void_p, c_void_p, c_void_p, c_int, c_longlong, c_void_p],
-        "mlb_bigram_add": [c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
+        "mlb_bigram_add": [c_void_p, c_void_p, c_int, c_void_p, c_int, c_float, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
                            c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
         "mlb_softcap_rows": [c_void_p, c_longlong, c_float, c_void_p],
     },
@@ -170,7 +170,7 @@ def part_sources():
     """(source, defines) of the kernels that only some kinds of parts ask for (each part names its own in
     `kernel_sources`)."""
     return [("residual.cu", {}), ("grouped_gemm.cu", {}), ("grouped_mma.cu", {}), ("latent.cu", {}), ("moe.cu", {}),
-            ("layernorm.cu", {}), ("short_conv.cu", {}), ("attention_kv.cu", {}), ("delta_rule.cu", {}),
+            ("layernorm.cu", {}), ("short_conv.cu", {}), ("state_space.cu", {}), ("attention_kv.cu", {}), ("delta_rule.cu", {}),
             ("linear_attention.cu", {}), ("post_norm.cu", {}), ("streams.cu", {})]
 
 
@@ -183,7 +183,7 @@ def all_sources():
         out += attention.mma_sources(d) + attention.tc_sources(d)
     from . import gemm_bf16, latent
     return (out + gemm_bf16.sources() + [("gemv_noalloc.cu", {})] + part_sources()
-            + latent.mma_sources(256, 32) + latent.mma_sources(512, 64))      # the widths of the presets
+            + latent.mma_sources(32, 8) + latent.mma_sources(256, 32) + latent.mma_sources(512, 64))      # the widths of the presets
 
 
 # ------------------------------------------------------------------------------ basic
@@ -422,7 +422,7 @@ def scale_add_layernorm(x: torch.Tensor, alpha: float, terms, weight: torch.Tens
 def normed_add_rmsnorm(x: torch.Tensor, terms, post_weight: torch.Tensor, eps: float, next_weight: Optional[torch.Tensor] = None,
                        out: Optional[torch.Tensor] = None) -> None:
     """d = sum_i s_i * d_i;  x += d / rms(d) * post_weight in place (fp32);  then, when `out` is given, out = x / rms(x) *
-    next_weight in out's dtype.  `terms`: one or two (s_i, d_i); a d_i may be [S, M, N] partial results, summed over S in order."""
+    next_weight in out's dtype, or without a `next_weight` x itself in out's dtype.  `terms`: one or two (s_i, d_i); a d_i may be [S, M, N] partial results, summed over S in order."""
     _need(x, "x", torch.float32, 2); _need(post_weight, "post_weight", torch.float32, 1)
     terms = list(terms)
     if not 1 <= len(terms) <= 2:
@@ -430,9 +430,11 @@ def normed_add_rmsnorm(x: torch.Tensor, terms, post_weight: torch.Tensor, eps: f
     if post_weight.shape[0] != x.shape[1]:
         raise KernelError("normed_add_rmsnorm: shapes do not agree")
     if out is not None:
-        _need(out, "out", dims=2); _need(next_weight, "next_weight", torch.float32, 1)
-        if out.shape != x.shape or next_weight.shape[0] != x.shape[1]:
-            raise KernelError("normed_add_rmsnorm: the normed copy must have the stream's shape")
+        _need(out, "out", dims=2)
+        if next_weight is not None:
+            _need(next_weight, "next_weight", torch.float32, 1)
+        if out.shape != x.shape or (next_weight is not None and next_weight.shape[0] != x.shape[1]):
+            raise KernelError("normed_add_rmsnorm: the copy must have the stream's shape")
     args = []
     for s, d in terms:
         n, stride = _partials(d, x.shape, "normed_add_rmsnorm term")
@@ -557,10 +559,10 @@ def stream_entry(x: torch.Tensor, x0: Optional[torch.Tensor], vector: torch.Tens
 
 
 def bigram_add(x: torch.Tensor, table: torch.Tensor, ctx, state: torch.Tensor, slots: torch.Tensor, buckets: int, mul_prev: int,
-               mul_cur: int, update_state: bool = True, token_table: Optional[torch.Tensor] = None) -> None:
+               mul_cur: int, update_state: bool = True, token_table: Optional[torch.Tensor] = None, scale: float = 1.0) -> None:
     """x[t] += table[(previous token * mul_prev + token * mul_cur) mod buckets], row `buckets` for a sequence's first token.
     The token in front of a step's first token is `state[slot]` ([slots, 1] int32), which then takes the step's last token.
-    With `token_table` [vocab, width] (the dtype of `table`): x[t] = token_table[token] + that row, in one pass."""
+    With `token_table` [vocab, width] (the dtype of `table`): x[t] = token_table[token] * scale + that row, in one pass."""
     if token_table is not None:
         _need(token_table, "token_table", table.dtype, 2)
         if token_table.shape[1] != x.shape[1]:
@@ -570,7 +572,7 @@ def bigram_add(x: torch.Tensor, table: torch.Tensor, ctx, state: torch.Tensor, s
         raise KernelError("bigram_add: the table has buckets + 1 rows of the stream's width, the state one int per slot")
     L = lib("residual.cu")
     build.check(L, L.mlb_bigram_add(x.data_ptr(), table.data_ptr(), dtype_tag(table), _ptr(token_table),
-                                    token_table.shape[0] if token_table is not None else 0, ctx.token_ids.data_ptr(), ctx.token_seq.data_ptr(),
+                                    token_table.shape[0] if token_table is not None else 0, float(scale), ctx.token_ids.data_ptr(), ctx.token_seq.data_ptr(),
                                     ctx.seq_starts.data_ptr(), ctx.seq_pos0.data_ptr(), state.data_ptr(), slots.data_ptr(), state.shape[0],
                                     x.shape[0], ctx.num_seqs, x.shape[1], int(buckets), int(mul_prev), int(mul_cur),
                                     1 if update_state else 0, _ptr(ctx.error_flag), _stream()))

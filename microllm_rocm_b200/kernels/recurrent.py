@@ -16,7 +16,7 @@ MAX_TAPS = 17
 MAX_WIDTH = 256
 
 ops.register_signatures("short_conv.cu", {
-    "mlb_short_conv": [c_void_p, c_longlong, c_int, c_longlong, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
+    "mlb_short_conv": [c_void_p, c_longlong, c_int, c_longlong, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
                        c_void_p, c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
     "mlb_short_conv_state": [c_void_p, c_longlong, c_int, c_longlong, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int,
                              c_int, c_void_p],
@@ -28,7 +28,7 @@ ops.register_signatures("delta_rule.cu", {
     "mlb_take_columns": [c_void_p, c_longlong, c_int, c_longlong, c_int, c_int, c_int, c_void_p, c_int, c_int, c_void_p],
     "mlb_linear_scan": [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int,
                         c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
-    "mlb_head_scan": [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
+    "mlb_head_scan": [c_void_p, c_void_p, c_longlong, c_int, c_void_p, c_int, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
                       c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
     "mlb_delta_scan": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
                        c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
@@ -46,8 +46,8 @@ def delta_sources():
 
 
 def short_conv(u: torch.Tensor, col0: int, weight: torch.Tensor, state: Optional[torch.Tensor], slots: torch.Tensor, ctx,
-               out: torch.Tensor, silu: bool, update_state: bool = True) -> None:
-    """out[t, c] = act(sum_j weight[c, j] * u[t - taps + 1 + j, col0 + c]) over the time of each sequence of the step
+               out: torch.Tensor, silu: bool, update_state: bool = True, bias: Optional[torch.Tensor] = None) -> None:
+    """out[t, c] = act(bias[c] + sum_j weight[c, j] * u[t - taps + 1 + j, col0 + c]) over the time of each sequence of the step
     `ctx`; inputs before the step come from `state` [slots, taps - 1, C] (zero before position 0).  Then the state
     moves on to hold the step's last inputs (unless `update_state` is False: a run that reads another run's state)."""
     _, ld, n, stride = _columns(u, "u")
@@ -56,6 +56,10 @@ def short_conv(u: torch.Tensor, col0: int, weight: torch.Tensor, state: Optional
     T = u.shape[-2]
     if out.shape != (T, C) or col0 < 0 or col0 + C > ld or not 1 <= taps <= MAX_TAPS:
         raise KernelError("short_conv: shapes do not agree")
+    if bias is not None:
+        ops._need(bias, "bias", torch.float32, 1)
+        if bias.shape[0] != C:
+            raise KernelError("short_conv: one bias per channel")
     num_slots = 1
     if taps > 1:
         ops._need(state, "state", torch.float32, 3)
@@ -63,7 +67,7 @@ def short_conv(u: torch.Tensor, col0: int, weight: torch.Tensor, state: Optional
             raise KernelError(f"short_conv: the state must be [slots, {taps - 1}, {C}], got {tuple(state.shape)}")
         num_slots = state.shape[0]
     L = ops.lib("short_conv.cu")
-    build.check(L, L.mlb_short_conv(u.data_ptr(), ld, n, stride, col0, weight.data_ptr(), ops._ptr(state), slots.data_ptr(), num_slots,
+    build.check(L, L.mlb_short_conv(u.data_ptr(), ld, n, stride, col0, weight.data_ptr(), ops._ptr(bias), ops._ptr(state), slots.data_ptr(), num_slots,
                                     ctx.seq_starts.data_ptr(), ctx.seq_pos0.data_ptr(), ctx.token_seq.data_ptr(), out.data_ptr(),
                                     out.shape[1], T, ctx.num_seqs, C, taps, 1 if silu else 0, ops._ptr(ctx.error_flag), ops._stream()))
     if taps > 1 and update_state:
@@ -186,15 +190,20 @@ def linear_scan(rule: str, q: torch.Tensor, k: torch.Tensor, decay: torch.Tensor
 
 def head_scan(q: torch.Tensor, k: torch.Tensor, decay: torch.Tensor, v: torch.Tensor, o: torch.Tensor, state: torch.Tensor,
               slots: torch.Tensor, ctx, heads: int, dk: int, dv: int, weight: Optional[torch.Tensor] = None,
-              n_state: Optional[torch.Tensor] = None, den: Optional[torch.Tensor] = None) -> None:
+              n_state: Optional[torch.Tensor] = None, den: Optional[torch.Tensor] = None, kv_heads: Optional[int] = None) -> None:
     """A recurrence with one decay per head over the step's tokens, per head with S [dk, dv]:
       S <- decay_t S + weight_t k_t v_t^T;  o_t = S^T q_t
     `decay` [T, heads], or [heads]: one fixed number per head; `weight` [T, heads] or None (1).  With `n_state`
     [slots, heads, dk] and `den` [T, heads] a vector runs beside S: n <- decay_t n + weight_t k_t, den_t = n . q_t.
-    q, k [T, heads * dk], v, o [T, heads * dv] fp32; states fp32, taken as zero for a sequence that starts at position 0."""
-    T = q.shape[0]
-    for name, t, shape in (("q", q, (T, heads * dk)), ("k", k, (T, heads * dk)), ("v", v, (T, heads * dv)), ("o", o, (T, heads * dv))):
-        ops._need(t, name, torch.float32, 2)
+    q, k [T, kv_heads * dk] (kv_heads None: heads; else head h reads q/k head h // (heads / kv_heads)), v, o [T, heads * dv] fp32;
+    q, k (of one row pitch) and v may be column views of wider rows; states fp32, taken as zero for a sequence that starts at position 0."""
+    T, G = q.shape[0], kv_heads or heads
+    ops._need(o, "o", torch.float32, 2)
+    if heads % G or q.stride(0) != k.stride(0):
+        raise KernelError("head_scan: heads must be a multiple of kv_heads, and q and k rows of one pitch")
+    for name, t, shape in (("q", q, (T, G * dk)), ("k", k, (T, G * dk)), ("v", v, (T, heads * dv)), ("o", o, (T, heads * dv))):
+        if not t.is_cuda or t.dtype != torch.float32 or t.dim() != 2 or t.stride(1) != 1:
+            raise KernelError(f"head_scan: {name} must be fp32 rows on the device")
         if tuple(t.shape) != shape:
             raise KernelError(f"head_scan: {name} must be {shape}, got {tuple(t.shape)}")
     per_token = decay.dim() == 2
@@ -213,7 +222,7 @@ def head_scan(q: torch.Tensor, k: torch.Tensor, decay: torch.Tensor, v: torch.Te
         if tuple(n_state.shape) != (state.shape[0], heads, dk):
             raise KernelError(f"head_scan: the vector's state must be [{state.shape[0]}, {heads}, {dk}], got {tuple(n_state.shape)}")
     L = ops.lib("delta_rule.cu")
-    build.check(L, L.mlb_head_scan(q.data_ptr(), k.data_ptr(), decay.data_ptr(), 1 if per_token else 0, ops._ptr(weight), v.data_ptr(), v.stride(0),
+    build.check(L, L.mlb_head_scan(q.data_ptr(), k.data_ptr(), q.stride(0), G, decay.data_ptr(), 1 if per_token else 0, ops._ptr(weight), v.data_ptr(), v.stride(0),
                                    o.data_ptr(), state.data_ptr(), ops._ptr(n_state), ops._ptr(den), slots.data_ptr(), state.shape[0],
                                    ctx.seq_starts.data_ptr(), ctx.seq_pos0.data_ptr(), ctx.num_seqs, heads, dk, dv, ops._ptr(ctx.error_flag),
                                    ops._stream()))

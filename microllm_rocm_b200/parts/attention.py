@@ -184,6 +184,7 @@ class NormedAttention(Mixer):
     Further options: `bias` (q and k projections have biases, added as the projection is read; values that are the projected
     keys carry the key's bias), `qk_norm="row"` (q and k are each divided by the root mean square of their WHOLE projection
     row, before the split into heads, times a weight of the row's length), `softcap` (score <- cap * tanh(score / cap)),
+    `keep_first` (with a window: the first tokens of a sequence stay visible in front of it),
     `distance_bias` {buckets, far} (score + R[bucket(query - key), head] with a learned table R of `buckets` rows: distances below
     buckets // 2 have a row each, from there on the rows widen logarithmically up to `far`; neither scaled nor capped),
     `sink` ("learned": one number per head whose exponential joins the softmax's denominator, with no key and no value,
@@ -222,6 +223,9 @@ class NormedAttention(Mixer):
             raise ValueError("normed_attention: a distance bias needs two rows or more and `far` beyond half of them")
         self.q_temp = tuple(params["q_temp"]) if params.get("q_temp") else None
         self.window = params.get("window")
+        self.keep_first = int(params.get("keep_first") or 0) if self.window else 0      # without a window every token is visible
+        if self.keep_first < 0:
+            raise ValueError("normed_attention: keep_first must not be negative")
         self.chunk = int(params["chunk"]) if params.get("chunk") else None
         self.norm_weight = bool(params.get("qk_norm_weight", True))
         self.norm_where = params.get("qk_norm_where", "before")
@@ -272,7 +276,8 @@ class NormedAttention(Mixer):
     # --- declarations -----------------------------------------------------------------
     def cache_need(self):
         from .base import CompositeNeed, FixedStateNeed
-        kv = PagedKVNeed(self.nkv, self.dk, self.window, value_dim=self.dv) if self.stored is None else PagedKVNeed(self.nkv, self.stored, self.window)
+        kv = (PagedKVNeed(self.nkv, self.dk, self.window, value_dim=self.dv, keep_first=self.keep_first) if self.stored is None
+              else PagedKVNeed(self.nkv, self.stored, self.window, keep_first=self.keep_first))
         if self.taps <= 1:
             return kv
         return CompositeNeed((("kv", kv), ("conv", FixedStateNeed((self.taps - 1, self.conv_cols), torch.float32))))
@@ -384,7 +389,7 @@ class NormedAttention(Mixer):
             return None
         rotary = None if self.freq is None else (self.freq.data_ptr(), self.rot_dims, self.magnitude)
         return ("normed_attention", self.hidden, self.nh, self.nkv, self.dk, self.dv, self.scale, self.eps, self.values, self.taps,
-                self.has_gate, self.qk_norm, self.norm_weight, self.norm_where, self.q_temp, self.window, self.chunk, rotary,
+                self.has_gate, self.qk_norm, self.norm_weight, self.norm_where, self.q_temp, self.window, self.keep_first, self.chunk, rotary,
                 self.gate_per_head, self.row_norm, self.has_bias, self.softcap, self.sink_kind, self.kv_shared, self.distance)
 
     def own_tensors(self):
@@ -439,26 +444,26 @@ class NormedAttention(Mixer):
             wide = o if (sv == self.dv and gate is None) else ctx.buffer("normed_attention.o_stored", (T, self.nh * sv), dt)
             attention_kernels.paged_attention(q, kv_view.pages, wide, ctx, kv_view.block_table, self.nh, self.nkv, sk, self.scale,
                                               self.window, beside_mma_products=gemm_bf16.gemv_preferred(x, self.w_o), chunk=self.chunk,
-                                              sink=self.sink, softcap=self.softcap or 0.0, bias=self.bias)
+                                              sink=self.sink, softcap=self.softcap or 0.0, bias=self.bias, keep_first=self.keep_first)
             if wide is not o:
                 attention_kv.gate_heads(wide, o, gate, self.conv_cols, self.nh, self.dv, sv, per_head=self.gate_per_head)
-        elif self.stored is not None and self.sink is None and not self.softcap and self.bias is None:
+        elif self.stored is not None and self.sink is None and not self.softcap and self.bias is None and not self.keep_first:
             # a page size the tensor-core kernels do not take: the plain kernel of one width
             wide = ctx.buffer("normed_attention.o_stored", (T, self.nh * sv), dt)
             attention_kernels.paged_attention(q, kv_view.pages, wide, ctx, kv_view.block_table, self.nh, self.nkv, sk, self.scale, self.window,
                                               chunk=self.chunk)
             attention_kv.gate_heads(wide, o, gate, self.conv_cols, self.nh, self.dv, sv, per_head=self.gate_per_head)
         elif self.stored is not None:
-            # the same with a sink, a cap or a distance bias: the plain kernel of two widths, told that both are the stored one
+            # the same with a sink, a cap, a distance bias or kept first tokens: the plain kernel of two widths, told that both are the stored one
             wide = ctx.buffer("normed_attention.o_stored", (T, self.nh * sv), dt)
             attention_kv.paged_attention_kv(q, kv_view.pages, wide, ctx.positions, ctx.token_seq, kv_view.block_table, kv_view.page_size,
                                             self.nh, self.nkv, sk, sv, self.scale, self.window, None, 0, flag, chunk=self.chunk,
-                                            sink=self.sink, softcap=self.softcap or 0.0, bias=self.bias)
+                                            sink=self.sink, softcap=self.softcap or 0.0, bias=self.bias, keep_first=self.keep_first)
             attention_kv.gate_heads(wide, o, gate, self.conv_cols, self.nh, self.dv, sv, per_head=self.gate_per_head)
         else:
             attention_kv.paged_attention_kv(q, kv_view.pages, o, ctx.positions, ctx.token_seq, kv_view.block_table, kv_view.page_size,
                                             self.nh, self.nkv, self.dk, self.dv, self.scale, self.window, gate, self.conv_cols, flag,
                                             chunk=self.chunk, gate_per_head=self.gate_per_head, sink=self.sink, softcap=self.softcap or 0.0,
-                                            bias=self.bias)
+                                            bias=self.bias, keep_first=self.keep_first)
         return linear(o, self.w_o, None, torch.float32, partials_ok=True, error_flag=flag,
                       alloc=lambda shape, dtype: ctx.buffer("normed_attention.out", shape, dtype))

@@ -62,12 +62,14 @@ class PagedKVNeed:
     ever read (pages behind it may be given back while the request lives); None: all keys.
     `dtype`: what the pages store; None: the runtime's compute dtype.  `value_dim`: width of a value when it
     differs from a key's (None: head_dim); a page then holds the keys of all kv heads [NKV, page_size, head_dim]
-    followed by the values [NKV, page_size, value_dim], which for equal widths is the same bytes as [2, NKV, page_size, D]."""
+    followed by the values [NKV, page_size, value_dim], which for equal widths is the same bytes as [2, NKV, page_size, D].
+    `keep_first`: the first tokens of a sequence stay readable in front of the window (their pages are not given back)."""
     num_kv_heads: int
     head_dim: int
     window: Optional[int] = None
     dtype: Optional[torch.dtype] = None
     value_dim: Optional[int] = None
+    keep_first: int = 0
 
 
 @dataclass(frozen=True)

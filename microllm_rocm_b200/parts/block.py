@@ -208,3 +208,46 @@ class SandwichResidualBlock(Block):
         ops.normed_add_rmsnorm(residual, terms, self.w_post1, self.eps, next_weight=self.ffn_norm.weight, out=normed2)
         ops.normed_add_rmsnorm(residual, [(1.0, self.feed_forward.forward(normed2, ctx))], self.w_post2, self.eps)
         return residual, None
+
+
+@register_block("output_norm_residual")
+class OutputNormResidualBlock(Block):
+    """A norm on every sublayer's result and none in front of it:  x += norm1(mixer(x));  x += norm2(feed_forward(x)).  The
+    sublayers read the stream itself, so the stream that leaves the block is final (no delta is handed on) and, on the bf16
+    path, travels with a bf16 copy for the products that read it; sums and norms are fp32.  A sublayer's result is added up
+    (partial sums, weighted terms of several mixers side by side), normalised and added, and the copy made, in ONE kernel."""
+    carries_no_delta = True
+
+    def __init__(self, params: dict, rt: Runtime, mixer_norm: Norm, mixer: Mixer, ffn_norm: Norm, feed_forward: FeedForward):
+        self.rt = rt
+        self.prefix = params.get("prefix", "")
+        self.mixer_norm, self.mixer, self.ffn_norm, self.feed_forward = mixer_norm, mixer, ffn_norm, feed_forward
+        self.has_ff = not getattr(feed_forward, "absent", False)
+        for norm in (mixer_norm, ffn_norm) if self.has_ff else (mixer_norm,):
+            if not hasattr(norm, "add_normed"):
+                raise TypeError("output_norm_residual needs norms that can add a normalised result in place (add_normed)")
+
+    def kernel_sources(self):
+        return [("post_norm.cu", {})]
+
+    def replay_key(self):
+        keys = [p.replay_key() for p in (self.mixer_norm, self.mixer, self.ffn_norm, self.feed_forward)]
+        return None if any(k is None for k in keys) else ("output_norm_residual", self.rt.dtype, *keys)
+
+    def own_tensors(self):
+        return [t for p in (self.mixer_norm, self.mixer, self.ffn_norm, self.feed_forward) for t in p.own_tensors()]
+
+    def forward(self, residual: torch.Tensor, delta: Optional[torch.Tensor], ctx: StepContext, cache):
+        if delta is not None:            # a block of another arrangement ran before this one
+            ops.add_inplace(residual, delta)
+        copy = None if self.rt.is_fp32 else ctx.buffer("block.stream_copy", tuple(residual.shape), self.rt.dtype)
+        x = residual if copy is None else copy
+        if copy is not None and (delta is not None or ctx.step_values.get("block.stream_copy_of") != residual.data_ptr()):
+            ops.cast_f32_bf16(residual, copy)                # the first block of a step: nobody has made the copy yet
+        terms = self.mixer.forward_terms(x, ctx, cache) if hasattr(self.mixer, "forward_terms") else [(1.0, self.mixer.forward(x, ctx, cache))]
+        self.mixer_norm.add_normed(residual, terms, copy)
+        if self.has_ff:
+            self.ffn_norm.add_normed(residual, [(1.0, self.feed_forward.forward(x, ctx))], copy)
+        if copy is not None:
+            ctx.step_values["block.stream_copy_of"] = residual.data_ptr()
+        return residual, None

@@ -136,7 +136,7 @@ class Model:
                 if name is not None:
                     needs = [self.cache_entries[f"{name}.{sub}"].need for sub in self.run_cache_parts[name]] \
                         if name in self.run_cache_parts else [self.cache_entries[name].need]
-                    group = tuple((type(need).__name__, getattr(need, "window", None), getattr(need, "dtype", None)) for need in needs)
+                    group = tuple((type(need).__name__, getattr(need, "window", None), getattr(need, "keep_first", 0), getattr(need, "dtype", None)) for need in needs)
                 keys.append(None if key is None else (key, owns, group))
             self._replay_keys = keys
         return self._replay_keys

@@ -25,7 +25,7 @@ class TokenEmbedding(Part):
         self.norm = (str(params["norm"][0]), float(params["norm"][1])) if params.get("norm") else None
         self.norm_weight: Optional[torch.Tensor] = None
         # a second table of buckets + 1 rows: row (previous token * mul_prev + token * mul_cur) mod buckets is added, the last
-        # row for a sequence's first token.  {"name", "buckets", "mul_prev", "mul_cur"} or None
+        # row for a sequence's first token (the multipliers only count modulo buckets, which keeps them small).  {"name", "buckets", "mul_prev", "mul_cur"} or None
         bg = params.get("bigram")
         self.bigram = dict(name=str(bg["name"]), buckets=int(bg["buckets"]), mul_prev=int(bg["mul_prev"]), mul_cur=int(bg["mul_cur"])) if bg else None
         if self.bigram and self.bigram["buckets"] <= 0:
@@ -70,7 +70,7 @@ class TokenEmbedding(Part):
         out = torch.empty((token_ids.shape[0], self.hidden), dtype=torch.float32, device=token_ids.device)
         if self.bigram and (ctx is None or state is None):
             raise RuntimeError("token_embedding: a pair table needs the step's context and the sequences' state")
-        one_pass = self.bigram and self.scale == 1.0 and self.bigram_table.dtype == self.table.dtype      # both rows gathered and added at once
+        one_pass = self.bigram and self.bigram_table.dtype == self.table.dtype      # both rows gathered and added at once
         if one_pass:
             pass
         elif self.scale != 1.0:
@@ -79,8 +79,8 @@ class TokenEmbedding(Part):
             ops.embed_gather(self.table, token_ids, out)
         if self.bigram:
             b = self.bigram
-            ops.bigram_add(out, self.bigram_table, ctx, state.storage, state.slots, b["buckets"], b["mul_prev"], b["mul_cur"],
-                           update_state=state.writable, token_table=self.table if one_pass else None)
+            ops.bigram_add(out, self.bigram_table, ctx, state.storage, state.slots, b["buckets"], b["mul_prev"] % b["buckets"], b["mul_cur"] % b["buckets"],
+                           update_state=state.writable, token_table=self.table if one_pass else None, scale=self.scale)
         if self.norm:
             ops.rmsnorm(out, self.norm_weight, self.norm[1], out)          # in place, fp32
         return out

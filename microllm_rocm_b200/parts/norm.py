@@ -1,4 +1,6 @@
-"""RMSNorm: y = x * (1 / sqrt(mean(x^2) + eps)) * w, all in fp32 (`one_plus`: the checkpoint stores w - 1, a weight around zero)
+"""RMSNorm: y = x * (1 / sqrt(mean(x^2) + eps)) * w, all in fp32 (`one_plus`: the checkpoint stores w - 1, a weight around zero;
+`scale`: a fixed factor on y, taken into the weight once).  Besides the plain form it offers the step of a block that
+normalises a sublayer's result before adding it: x += norm(weighted results), in place
 (reference: src/ops/ops.cpp:684-699; fused with the residual add at :702-740).
 LayerNorm: y = (x - mean) / sqrt(mean((x - mean)^2) + eps) * w + b, all in fp32 (`bias=False`: no b); besides the plain form it offers the
 step of a block that normalises AFTER its sums: x <- norm(alpha * x + weighted results), in place."""
@@ -21,6 +23,7 @@ class RMSNorm(Norm):
         self.name = params.get("name", "weight")         # the weight's local name in the checkpoint
         self.absent = bool(params.get("absent", False))  # a norm in front of a sub-layer that the layer leaves out: no weight, never run
         self.one_plus = bool(params.get("one_plus", False))   # the stored tensor is the weight minus one: 1 is added once, at bind, in fp32
+        self.scale = float(params.get("scale", 1.0))
         self.rt = rt
         self.weight: Optional[torch.Tensor] = None
 
@@ -33,6 +36,8 @@ class RMSNorm(Norm):
         self.weight = tensors.get(self.name) if self.absent else tensors[self.name]
         if self.one_plus and self.weight is not None:
             self.weight = (self.weight.to(torch.float32) + 1.0).contiguous()
+        if self.scale != 1.0 and self.weight is not None:
+            self.weight = (self.weight.to(torch.float32) * self.scale).contiguous()
 
     def replay_key(self):
         return ("rmsnorm", self.size, self.eps)
@@ -53,6 +58,10 @@ class RMSNorm(Norm):
             ops.add_scaled_rmsnorm(residual, delta, scale, self.weight, self.eps, out)
         else:
             ops.add_rmsnorm(residual, delta, self.weight, self.eps, out)
+
+    def add_normed(self, stream: torch.Tensor, terms, copy: Optional[torch.Tensor]) -> None:
+        """stream += norm(sum_i s_i * d_i) in place (fp32); `copy` receives the new stream in its dtype."""
+        ops.normed_add_rmsnorm(stream, terms, self.weight, self.eps, out=copy)
 
 
 @register_norm("layernorm")

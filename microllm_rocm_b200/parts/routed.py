@@ -9,7 +9,9 @@
 a tensor named by `router_bias_name`, only steers the choice) and the weights are the chosen s themselves, not renormalised.
 `scoring="sigmoid_groups"` with `groups`, `keep`, `weight_scale`: s = sigmoid(z); the experts form equal groups of neighbours, a
 group scores the sum of its two largest s, only experts of the `keep` best groups can be chosen; the weights are the chosen s
-divided by their sum, times `weight_scale`.  `activation="clamped_swish"` with `limit`: the experts' inner activation is the
+divided by their sum, times `weight_scale`.  `scoring="sigmoid"`: s = sigmoid(z), the `top` largest run with the chosen s times
+`weight_scale` as they are.  `weight_on="input"`: an expert gets w * x instead of x and its result is added as it is (both of its
+first products are multiplied by w in fp32, which is the same thing).  `activation="clamped_swish"` with `limit`: the experts' inner activation is the
 clamped form of the dense feed-forward.
 `identity` = n: the router has experts + n outputs, and the last n have no expert behind them: a token that chooses one gets
 its own input back, times the weight.
@@ -60,8 +62,11 @@ class RoutedExperts(FeedForward):
             if self.identity or self.groups <= 0 or self.experts % self.groups or not 0 < self.keep <= self.groups \
                     or self.top > self.keep * (self.experts // self.groups):
                 raise ValueError(f"routed experts: top {self.top} of {self.keep} of {self.groups} groups of {self.experts} experts")
-        elif self.groups != 1 or self.weight_scale != 1.0:
-            raise ValueError(f"routed experts: scoring {self.scoring!r} has neither groups nor a factor on the weights")
+        elif self.groups != 1 or (self.weight_scale != 1.0 and self.scoring != "sigmoid"):
+            raise ValueError(f"routed experts: scoring {self.scoring!r} has no groups, and only sigmoid scores a factor on the weights")
+        self.weight_on = params.get("weight_on", "output")
+        if self.weight_on not in ("output", "input") or (self.weight_on == "input" and self.identity):
+            raise ValueError(f"routed experts: weight_on {self.weight_on!r} (with {self.identity} outputs that pass the input on)")
         self.activation = params.get("activation", "silu")
         self.limit = float(params["limit"]) if params.get("limit") is not None else None
         if self.activation not in ("silu", CLAMPED_ACTIVATION) or (self.activation == CLAMPED_ACTIVATION and not (self.limit or 0) > 0):
@@ -150,7 +155,7 @@ class RoutedExperts(FeedForward):
         if not self.rt.is_fp32 and not gemm_bf16._direct_library(self.rt.device):
             return None                  # the library product would go through the tensor framework
         return ("routed_experts", self.hidden, self.experts, self.top, self.inter, shared, self.has_gate, self.b_router is not None,
-                self.scoring, self.identity, self.groups, self.keep, self.weight_scale, self.activation, self.limit)
+                self.scoring, self.identity, self.groups, self.keep, self.weight_scale, self.activation, self.limit, self.weight_on)
 
     def own_tensors(self):
         own = [self.w_gate_up, self.w_down, self.w_router, self.b_router]
@@ -173,17 +178,25 @@ class RoutedExperts(FeedForward):
                    groups=self.groups, keep=self.keep, weight_scale=self.weight_scale)
         offsets = buf("offsets", (E + 1,), torch.int32)
         order = buf("order", (P,), torch.int32)
-        moe.align(ids, E, offsets, order, flag, passthrough=self.identity)
+        # weights that went in leave nothing but a sum: the experts' results are then the delta's partial sums, one per choice, and
+        # whoever takes the delta in adds them up (no pass of its own)
+        weigh_in = self.weight_on == "input"
+        partials = weigh_in and self.shared is None and out_scale is None
+        dest = buf("dest", (P,), torch.int32) if partials and top > 1 else None
+        moe.align(ids, E, offsets, order, flag, passthrough=self.identity, dest=dest)
         row_tile = grouped.row_tile_for(P, E, True, grouped.mma_supported(x, self.w_gate_up))
         act = buf("act", (P, ff), self.rt.dtype)
         grouped.grouped_silu_mul(x, self.w_gate_up, act, rows=P, group_offsets=offsets, a_rows=order, a_row_div=top,
-                                 row_tile=row_tile, alloc=lambda shape, dtype: buf("gate_up", shape, dtype), activation=self.activation, limit=self.limit)
+                                 row_tile=row_tile, alloc=lambda shape, dtype: buf("gate_up", shape, dtype), activation=self.activation, limit=self.limit,
+                                 row_scale=weights.view(-1) if weigh_in else None)
         y = buf("y", (P, W), torch.float32)
-        grouped.grouped_linear(act, self.w_down, y, rows=P, group_offsets=offsets, c_rows=order, row_tile=row_tile)
+        grouped.grouped_linear(act, self.w_down, y, rows=P, group_offsets=offsets, c_rows=order if dest is None else dest, row_tile=row_tile)
+        if partials:
+            return y.view(top, T, W) if top > 1 else y
         shared = self.shared.forward(x, ctx) if self.shared is not None else None
         out = buf("out", (T, W), torch.float32)
         if self.identity:
             moe.combine(y, weights, out, shared=shared, gate=gate, col_scale=out_scale, ids=ids, experts=E, x=x)
         else:
-            moe.combine(y, weights, out, shared=shared, gate=gate, col_scale=out_scale)
+            moe.combine(y, None if weigh_in else weights, out, shared=shared, gate=gate, col_scale=out_scale, top=top)
         return out
