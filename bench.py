@@ -324,6 +324,12 @@ def step_timeline(session):
 # same width, layers and vocabulary: an attention layer with the same heads where Gubidra has one, a parallel layer (those
 # attention heads beside linear attention with the recurrence's heads and widths) where Gubidra has a recurrence, and routed
 # experts of the same count and width.
+# The Naburax sizes (a scaled pair-table embedding; a norm on every sublayer's result and none in front; a layer of windowed
+# attention with kept first tokens beside a selective state space, then latent attention whose queries have a latent of their
+# own, one windowed; routed experts whose weights multiply their input) stand beside the two closest designs that were here
+# before, both of the same width, layer count and vocabulary with routed experts of the same count and width: a Gedalix whose
+# latent attention has the same heads and widths in every layer, and a Gubidra that alternates retention with the state space's
+# heads and widths and windowed attention with the attention branch's.
 DESIGN_SIZES = {
     "small": dict(gedalix="gedalix-small", layers=4),
     "16b-layers": dict(gedalix="gedalix-16b-layers", layers=4),
@@ -335,6 +341,8 @@ DESIGN_SIZES = {
     "lozepel-3b-layers": dict(lozepel="lozepel-3b-layers", layers=4),
     "gubidra-small": dict(gubidra="gubidra-small", layers=4),
     "gubidra-3b-layers": dict(gubidra="gubidra-3b-layers", layers=4),
+    "naburax-small": dict(naburax="naburax-small", layers=4),
+    "naburax-3b-layers": dict(naburax="naburax-3b-layers", layers=4),
 }
 
 
@@ -407,6 +415,26 @@ def _equal_lozepel_gubidra(raw, layers, max_positions):
                                     "layers": made, "max_positions": max_positions})
 
 
+def _equal_gedalix_naburax(raw, layers, max_positions):
+    from microllm_rocm_b200.config.gedalix import GedalixConfig, _layer
+    one = next(l for l in raw["layers"] if l["type"] == "latent_attention")
+    m, r = one["mixer"], one["mlp"]
+    layer = _layer(m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"], r["router"]["experts"], r["router"]["top"], r["expert"]["ff"], None)
+    return GedalixConfig.from_dict({"architecture": "Gedalix", "vocab": raw["vocab"], "width": raw["width"], "max_positions": max_positions,
+                                    "embedding": {"scale": 4.0}, "norm": {"eps": 1e-6}, "residual_mult": 0.5, "layers": [layer] * layers})
+
+
+def _equal_gubidra_naburax(raw, layers, max_positions):
+    from microllm_rocm_b200.config.gubidra import GubidraConfig, attention_layer, moe, retention_layer
+    par = next(l for l in raw["layers"] if l["type"] == "parallel")
+    left, right, r = par["mixer"]["left"], par["mixer"]["right"], par["mlp"]
+    ff = moe(r["router"]["experts"], r["router"]["top"], r["expert"]["ff"])
+    made = [retention_layer(right["heads"], right["state"], right["vdim"], ff),
+            attention_layer(left["heads"], left["kv_heads"], left["dim"], left["vdim"], left["mask"]["size"], ff)]
+    return GubidraConfig.from_dict({"architecture": "Gubidra", "vocab": raw["vocab"], "width": raw["width"], "streams": 2, "embedding": {"scale": 4.0},
+                                    "norm": {"eps": 1e-5}, "layers": [made[i % 2] for i in range(layers)], "max_positions": max_positions})
+
+
 def _kernel_rows(step_fn, repeats=3):
     """(name, launches, summed duration in us, summed exposed time in us: see _exposed) of one call of step_fn, the
     kernels that add most to the step first.  Kernels start early behind their predecessors, so a duration holds
@@ -423,7 +451,7 @@ def _kernel_rows(step_fn, repeats=3):
         row[0] += 1
         row[1] += duration
         row[2] += exposed
-    return [(n, c, round(d, 1), round(e, 1)) for n, (c, d, e) in sorted(rows.items(), key=lambda kv: -kv[1][2])][:20]
+    return [(n, c, round(d, 1), round(e, 1)) for n, (c, d, e) in sorted(rows.items(), key=lambda kv: -kv[1][2])][:28]
 
 
 def run_designs(args):
@@ -442,7 +470,14 @@ def run_designs(args):
     for name in names:
         size = DESIGN_SIZES[name]
         layers = args.layers or size["layers"]
-        if "gubidra" in size:
+        if "naburax" in size:
+            from microllm_rocm_b200.config.naburax import PRESETS as NABURAX_PRESETS, NaburaxConfig
+            raw = copy.deepcopy(NABURAX_PRESETS[size["naburax"]])
+            raw["layers"] = raw["layers"][:layers]
+            raw["max_positions"] = args.prompt + 512
+            designs = {"naburax": NaburaxConfig.from_dict(raw), "gedalix": _equal_gedalix_naburax(raw, layers, args.prompt + 512),
+                       "gubidra": _equal_gubidra_naburax(raw, layers, args.prompt + 512)}
+        elif "gubidra" in size:
             from microllm_rocm_b200.config.gubidra import PRESETS as GUBIDRA_PRESETS, GubidraConfig
             raw = copy.deepcopy(GUBIDRA_PRESETS[size["gubidra"]])
             raw["layers"] = raw["layers"][:layers]

@@ -9,6 +9,8 @@
 //                 two largest s[e] + b[e] and only experts of the `keep` best groups can be chosen; the `top` largest of those
 //                 run with weights s / (sum of the chosen s + 1e-20) * weight_scale.
 //                 `scoring` 3: the same with the chosen s * weight_scale as the weights, not divided by their sum.
+//                 Without groups and correction the choice goes by the logits, which order the experts as their scores do but stay
+//                 apart where scores round to 1 (or 0).
 //   moe_align     (below) skips, without raising the flag, ids in [experts, experts + passthrough): outputs of the router that
 //                 have no expert behind them (moe_combine adds the token's own input times the weight for those).
 //   moe_align     from ids[T*top] to a list of the pairs (token, choice) sorted by expert: offsets[E+1] and
@@ -53,7 +55,7 @@ moe_select_kernel(const float* __restrict__ logits, long long ld, int n_partials
         for (int e = lane; e < experts; e += 32) {      // (every lane turns its own elements)
             const float v = z[e], sc = v >= 0.0f ? 1.0f / (1.0f + expf(-v)) : expf(v) / (1.0f + expf(v));
             score[e] = sc;
-            z[e] = sc + (bias ? bias[e] : 0.0f);
+            if (scoring == 2 || bias || keep < groups) z[e] = sc + (bias ? bias[e] : 0.0f);
         }
         __syncwarp();
         if (keep < groups) {

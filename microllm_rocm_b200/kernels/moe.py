@@ -38,7 +38,8 @@ def select(logits: torch.Tensor, experts: int, bias: Optional[torch.Tensor], top
     s = sigmoid of every column; the experts form `groups` equal groups of neighbours, a group scores the sum of its two largest
     s + bias, only experts of the `keep` best groups can be chosen (ties: the smaller index), and the weights are the chosen s
     divided by their sum + 1e-20, times `weight_scale`.  "sigmoid": the same choice, the weights are the chosen s times
-    `weight_scale`, not divided by their sum."""
+    `weight_scale`, not divided by their sum; without groups and bias the choice goes by the logits themselves (the same order, but
+    scores that round to 1 stay apart)."""
     if scoring not in SCORINGS:
         raise KernelError(f"moe.select: scoring {scoring!r} is not one of {', '.join(SCORINGS)}")
     n_partials, stride, first = 1, 0, logits

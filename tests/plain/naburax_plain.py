@@ -85,12 +85,12 @@ def softmax_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, scale: 
     """q [T, H, dk], k [T, G, dk], v [T, G, dv]; query head h reads key/value head h // (H / G).  [T, H, dv]."""
     T, H, G = q.shape[0], q.shape[1], k.shape[1]
     out = torch.zeros((T, H, v.shape[-1]), dtype=F)
+    of_head = [h // (H // G) for h in range(H)]
+    k, v = k[:, of_head], v[:, of_head]                                          # [T, H, .]: every query head's own copy
     for i in range(T):
         seen = visible(i, window, keep_first)
-        for h in range(H):
-            g = h // (H // G)
-            p = torch.softmax((k[seen, g] @ q[i, h]) * scale, 0)
-            out[i, h] = p @ v[seen, g]
+        p = torch.softmax((k[seen] * q[i]).sum(-1) * scale, 0)                  # [seen, H]
+        out[i] = (p[:, :, None] * v[seen]).sum(0)
     return out
 
 
@@ -171,9 +171,10 @@ def mixer_latent(m: dict, w: Dict[str, torch.Tensor], p: str, h: torch.Tensor, e
 
 # ---------------------------------------------------------------------------------------- feed-forward
 def route(z: torch.Tensor, top: int):
-    """z [T, E] -> (chosen [T, top], their weights): sigmoid scores as they are (ties: the smaller index)."""
+    """z [T, E] -> (chosen [T, top], their weights): sigmoid scores as they are.  The sigmoid grows with z, so the largest z are the
+    largest scores, also where a score can no longer be told from 1 (ties: the smaller index)."""
     s = torch.sigmoid(z)
-    chosen = torch.tensor([sorted(range(z.shape[1]), key=lambda e: (-float(s[t, e]), e))[:top] for t in range(z.shape[0])])
+    chosen = torch.tensor([sorted(range(z.shape[1]), key=lambda e: (-float(z[t, e]), e))[:top] for t in range(z.shape[0])])
     return chosen, torch.gather(s, 1, chosen)
 
 
