@@ -66,51 +66,85 @@ __device__ __forceinline__ float proj_at(const PrepareParams& p, size_t row_base
 
 constexpr int SLICE = 1024;        // query and gate columns per block
 
-// The token's cache row: the normalised latent, then the shared key part with its rotation.
-template <typename KVT>
-__device__ __forceinline__ void store_cache_row(const PrepareParams& p, int t, size_t row, int pos, float* scratch) {
-    const int half = p.rot_dims / 2;
-    const int Dk = p.rank + p.rot_dim;
-    KVT* cache_row = nullptr;
-    if (p.pages) {
-        const int block = pos / p.page_size;
-        const int page = block < p.max_blocks ? p.block_table[(size_t)p.token_seq[t] * p.max_blocks + block] : -1;
-        if (page < 0 || page >= p.num_pages) {
-            if (threadIdx.x == 0 && p.error_flag) atomicExch(p.error_flag, 1);
-        } else {
-            cache_row = (KVT*)p.pages + ((size_t)page * p.page_size + pos % p.page_size) * Dk;
-        }
-        // the latent, divided by its root mean square, times the norm's weight
-        float ss = 0.0f;
-        for (int c = threadIdx.x; c < p.rank; c += blockDim.x) {
-            const float v = proj_at(p, row, p.kv_col + c);
-            ss += v * v;
-        }
-        ss = block_sum(ss, scratch);
-        const float inv = 1.0f / sqrtf(ss / (float)p.rank + p.eps);
-        if (cache_row) {
-            for (int c = threadIdx.x; c < p.rank; c += blockDim.x)
-                cache_row[c] = from_f32<KVT>(proj_at(p, row, p.kv_col + c) * inv * p.norm_weight[c]);
-            // the shared key part: its first rot_dims elements turned in pairs, the rest passed on
-            for (int i = threadIdx.x; i < p.rot_dim; i += blockDim.x) {
-                float out;
-                const float v = proj_at(p, row, p.kv_col + p.rank + i);
-                if (i < p.rot_dims) {
-                    const Pair pr = pair_of(i, half, p.interleaved);
-                    out = turned(v, proj_at(p, row, p.kv_col + p.rank + pr.other), pr.first, (float)pos * p.inv_freq[pr.index], p.magnitude);
-                } else {
-                    out = v;
-                }
-                cache_row[p.rank + i] = from_f32<KVT>(out);
-            }
+// A block's share of a row's norm: up to ROW_PER elements a thread stay in registers, fetched side by side (the partial results of
+// all of them a step of the sum at a time), so that a decode step's few rows pay one trip to memory; longer rows are read twice.
+constexpr int ROW_PER = 4;
+template <typename OutT>
+__device__ __forceinline__ void normed_row(const PrepareParams& p, size_t row, long long col, int n, const float* __restrict__ weight,
+                                           const float (&w)[ROW_PER], const float (&v)[ROW_PER], float* scratch, OutT* out) {
+    float ss = 0.0f;
+#pragma unroll
+    for (int i = 0; i < ROW_PER; ++i) ss = fmaf(v[i], v[i], ss);                   // (zero beyond the row)
+    for (int c = threadIdx.x + ROW_PER * blockDim.x; c < n; c += blockDim.x) { const float u = proj_at(p, row, col + c); ss = fmaf(u, u, ss); }
+    const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)n + p.eps);
+    if (!out) return;
+#pragma unroll
+    for (int i = 0; i < ROW_PER; ++i) {
+        const int c = threadIdx.x + i * blockDim.x;
+        if (c < n) out[c] = from_f32<OutT>(v[i] * inv * w[i]);
+    }
+    for (int c = threadIdx.x + ROW_PER * blockDim.x; c < n; c += blockDim.x) out[c] = from_f32<OutT>(proj_at(p, row, col + c) * inv * weight[c]);
+}
+__device__ __forceinline__ void fetch_row(const PrepareParams& p, size_t row, long long col, int n, float (&v)[ROW_PER]) {
+#pragma unroll
+    for (int i = 0; i < ROW_PER; ++i) {
+        const int c = threadIdx.x + i * blockDim.x;
+        v[i] = c < n ? p.proj[row + col + c] : 0.0f;
+    }
+#pragma unroll 4
+    for (int k = 1; k < p.n_partials; ++k) {
+        const float* const at = p.proj + (size_t)k * p.partial_stride + row + col;
+#pragma unroll
+        for (int i = 0; i < ROW_PER; ++i) {
+            const int c = threadIdx.x + i * blockDim.x;
+            if (c < n) v[i] += at[c];
         }
     }
+}
+__device__ __forceinline__ void fetch_weight(const float* __restrict__ weight, int n, float (&w)[ROW_PER]) {
+#pragma unroll
+    for (int i = 0; i < ROW_PER; ++i) {
+        const int c = threadIdx.x + i * blockDim.x;
+        w[i] = weight && c < n ? weight[c] : 0.0f;
+    }
+}
+
+// The token's cache row: the normalised latent, and behind it the shared key part with its rotation.  `w`: the norm's weights of
+// this thread (fetched before the wait for the predecessor).
+template <typename KVT>
+__device__ __forceinline__ void store_cache_row(const PrepareParams& p, int t, size_t row, int pos, const float (&w)[ROW_PER], float* scratch) {
+    if (!p.pages) return;
+    const int half = p.rot_dims / 2;
+    const int Dk = p.rank + p.rot_dim;
+    float v[ROW_PER];
+    fetch_row(p, row, p.kv_col, p.rank, v);
+    KVT* cache_row = nullptr;
+    const int block = pos / p.page_size;
+    const int page = block < p.max_blocks ? p.block_table[(size_t)p.token_seq[t] * p.max_blocks + block] : -1;
+    if (page < 0 || page >= p.num_pages) {
+        if (threadIdx.x == 0 && p.error_flag) atomicExch(p.error_flag, 1);
+    } else {
+        cache_row = (KVT*)p.pages + ((size_t)page * p.page_size + pos % p.page_size) * Dk;
+        // the shared key part: its first rot_dims elements turned in pairs, the rest passed on
+        for (int i = threadIdx.x; i < p.rot_dim; i += blockDim.x) {
+            float out = proj_at(p, row, p.kv_col + p.rank + i);
+            if (i < p.rot_dims) {
+                const Pair pr = pair_of(i, half, p.interleaved);
+                out = turned(out, proj_at(p, row, p.kv_col + p.rank + pr.other), pr.first, (float)pos * p.inv_freq[pr.index], p.magnitude);
+            }
+            cache_row[p.rank + i] = from_f32<KVT>(out);
+        }
+    }
+    normed_row(p, row, p.kv_col, p.rank, p.norm_weight, w, v, scratch, cache_row);
 }
 
 template <typename QT, typename KVT>
 __global__ void __launch_bounds__(256)
 latent_prepare_kernel(PrepareParams p) {
-    pdl_prologue();
+    pdl_launch_dependents();
+    float w[ROW_PER];
+    fetch_weight(p.pages && blockIdx.y == 0 ? p.norm_weight : nullptr, p.rank, w);
+    pdl_wait();
     __shared__ float scratch[32];
     const int t = blockIdx.x;
     const size_t row = (size_t)t * p.ld;
@@ -148,29 +182,28 @@ latent_prepare_kernel(PrepareParams p) {
         }
         return;
     }
-    store_cache_row<KVT>(p, t, row, pos, scratch);
+    store_cache_row<KVT>(p, t, row, pos, w, scratch);
 }
 
 // One block per token and part: blockIdx.y 0 the cache row, 1 the queries' latent.
+constexpr int COMPRESS_THREADS = 128;
 template <typename QT, typename KVT>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(COMPRESS_THREADS)
 latent_compress_kernel(PrepareParams p) {
-    pdl_prologue();
+    pdl_launch_dependents();
     __shared__ float scratch[32];
     const int t = blockIdx.x;
     const size_t row = (size_t)t * p.ld;
+    float w[ROW_PER];
+    fetch_weight(blockIdx.y == 0 ? p.norm_weight : p.cq_weight, blockIdx.y == 0 ? p.rank : p.cq_rank, w);
+    pdl_wait();
     if (blockIdx.y == 0) {
-        store_cache_row<KVT>(p, t, row, p.positions[t], scratch);
+        store_cache_row<KVT>(p, t, row, p.positions[t], w, scratch);
         return;
     }
-    float ss = 0.0f;
-    for (int c = threadIdx.x; c < p.cq_rank; c += blockDim.x) {
-        const float v = proj_at(p, row, p.cq_col + c);
-        ss = fmaf(v, v, ss);
-    }
-    const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)p.cq_rank + p.eps);
-    for (int c = threadIdx.x; c < p.cq_rank; c += blockDim.x)
-        ((QT*)p.cq_out)[(size_t)t * p.cq_rank + c] = from_f32<QT>(proj_at(p, row, p.cq_col + c) * inv * p.cq_weight[c]);
+    float v[ROW_PER];
+    fetch_row(p, row, p.cq_col, p.cq_rank, v);
+    normed_row(p, row, p.cq_col, p.cq_rank, p.cq_weight, w, v, scratch, (QT*)p.cq_out + (size_t)t * p.cq_rank);
 }
 
 constexpr int WARPS = 4;
@@ -310,9 +343,9 @@ MLB_EXPORT int mlb_latent_compress(const float* proj, long long ld, int n_partia
     p.tokens = tokens; p.rot_dim = rot_dim; p.rank = rank; p.error_flag = error_flag;
     p.cq_col = cq_col; p.cq_rank = cq_rank; p.cq_weight = cq_weight; p.cq_out = cq_out;
     const dim3 grid(tokens, 2);
-    if (q_dtype == MLB_F32 && (kv_dtype == MLB_F32 || !pages)) launch_kernel(latent_compress_kernel<float, float>, grid, 256, 0, stream, p);
+    if (q_dtype == MLB_F32 && (kv_dtype == MLB_F32 || !pages)) launch_kernel(latent_compress_kernel<float, float>, grid, COMPRESS_THREADS, 0, stream, p);
     else if (q_dtype == MLB_BF16 && (kv_dtype == MLB_BF16 || !pages))
-        launch_kernel(latent_compress_kernel<__nv_bfloat16, __nv_bfloat16>, grid, 256, 0, stream, p);
+        launch_kernel(latent_compress_kernel<__nv_bfloat16, __nv_bfloat16>, grid, COMPRESS_THREADS, 0, stream, p);
     else return fail(MLB_INVALID_ARGUMENT, "latent_compress: unsupported dtypes %d / %d", q_dtype, kv_dtype);
     return check_launch("latent_compress");
 }
