@@ -110,7 +110,7 @@ def left_attention(m: dict, w: Dict[str, torch.Tensor], p: str, h: torch.Tensor,
 
 # ---------------------------------------------------------------------------------------- selective state space
 def causal_conv(u: torch.Tensor, taps: torch.Tensor, bias: torch.Tensor) -> torch.Tensor:
-    """u [T, C], taps [C, n] (the last column is the current token's), zeros before the start."""
+    """u [T, C], taps [C, n]: out_t = bias + sum_j taps[:, n - 1 - j] u_(t-j), where u_i = 0 for i < 0."""
     n = taps.shape[1]
     padded = torch.cat([torch.zeros((n - 1, u.shape[1]), dtype=F), u], 0)
     out = torch.zeros_like(u) + bias.to(F)
